@@ -43,6 +43,8 @@ SYMBOLS = {
     "b200p_model_load": (_vp, [C.c_char_p, _vp]),
     "b200p_model_weights_of": (_vp, [_vp]),
     "b200p_model_free": (None, [_vp]),
+    "b200p_model_create": (_vp, [C.c_char_p, _i, _vp, _vp, _vp, _vp, _vp, _vp]),
+    "b200p_model_describe": (_i, [_vp, _vp, _i, _vp]),
     "b200p_attn_decode_workspace_bytes": (_sz, [_vp]),
     "b200p_attn_decode": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _sz, _vp]),
     "b200p_attn_decode_dyn": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _i, _vp, _sz, _vp]),
@@ -58,6 +60,9 @@ SYMBOLS = {
     "b200p_attn_prefill_debug": (_i, [_vp, _vp, _vp, _vp, _vp, _i, _vp, _vp]),
     "b200p_device_status": (_i, [_i]),
     "b200p_session_create": (_vp, [_vp, _i, _i, _vp]),
+    "b200p_session_open": (_vp, [_vp, _i, _i, _i, _vp]),
+    "b200p_session_extend": (_i, [_vp, _vp, _i, _vp, _i, _vp, _vp]),
+    "b200p_session_reset": (None, [_vp]),
     "b200p_session_destroy": (None, [_vp]),
     "b200p_session_generate": (_i, [_vp, _vp, _i, _i, _vp, _vp, _vp]),
     "b200p_session_prefill_logits": (_i, [_vp, _vp, _i, _vp, _vp]),
@@ -117,16 +122,25 @@ _lib = None
 def lib() -> C.CDLL:
     """libb200p.so, loaded once.  Raises if it has not been built (python
     amd-incstinct-labs_b200/build.py, or __graft_entry__.build())."""
-    global _lib
     if _lib is None:
         if not os.path.exists(LIB_PATH):
             raise RuntimeError(f"{LIB_PATH} is missing: build the CUDA library first; there is no fallback path")
-        h = C.CDLL(LIB_PATH)
-        for name, (res, args) in SYMBOLS.items():
-            fn = getattr(h, name)          # AttributeError if the library lacks a declared symbol
-            fn.restype, fn.argtypes = res, args
-        _lib = h
+        load_library(LIB_PATH)
     return _lib
+
+
+def load_library(path: str, whole: bool = True) -> C.CDLL:
+    """Use the library at `path`.  whole=False: one that holds a single decoder of the runtime (build.build_decoder),
+    with the entry points that it has."""
+    global _lib
+    h = C.CDLL(path)
+    for name, (res, args) in SYMBOLS.items():
+        if not whole and not hasattr(h, name):
+            continue
+        fn = getattr(h, name)              # AttributeError if the library lacks a declared symbol
+        fn.restype, fn.argtypes = res, args
+    _lib = h
+    return h
 
 
 def _check(status: int, where: str) -> None:
@@ -544,19 +558,44 @@ def read_model_meta(model_dir: str):
 
 
 class Model:
-    """A model directory (meta.json + per-tensor .bin files, cdna3::runtime::ModelLoader) loaded into
-    device memory the object owns."""
+    """A model in device memory the object owns: a directory in the reference's export format (meta.json + per-tensor
+    .bin files, cdna3::runtime::ModelLoader), or one with config.json + model.safetensors, whose "architecture" is
+    looked up in the library's registry.  from_tensors makes the latter from tensors on the device."""
 
     def __init__(self, model_dir: str):
         st = _i(0)
-        self._h = lib().b200p_model_load(os.fsencode(model_dir), C.byref(st))
-        if not self._h:
-            raise B200PError(st.value, "model_load")
-        self.weights = C.cast(lib().b200p_model_weights_of(self._h), C.POINTER(ModelWeights)).contents
-        self.cfg = {n: getattr(self.weights.cfg, n) for n, _ in ModelConfig._fields_}
+        self._adopt(lib().b200p_model_load(os.fsencode(model_dir), C.byref(st)), st, "model_load")
+
+    @classmethod
+    def from_tensors(cls, config: dict, tensors: dict):
+        """config: what config.json would hold; tensors: name -> contiguous CUDA tensor (kept alive)."""
+        import json
+        self = cls.__new__(cls)
+        names = list(tensors)
+        for n in names:
+            _dev(tensors[n], n)
+        self._tensors = dict(tensors)
+        dims = [d for n in names for d in tensors[n].shape]
+        k = len(names)
+        st = _i(0)
+        self._adopt(lib().b200p_model_create(
+            json.dumps(config).encode(), k, (C.c_char_p * k)(*[n.encode() for n in names]), (_vp * k)(*[tensors[n].data_ptr() for n in names]),
+            (_i * k)(*[_dtype_code(tensors[n]) for n in names]), (_i * k)(*[tensors[n].dim() for n in names]), (_ll * len(dims))(*dims),
+            C.byref(st)), st, "model_create")
+        return self
+
+    def _adopt(self, handle, status, where):
+        self._h = handle
+        if not handle:
+            raise B200PError(status.value, where)
+        mc, name = ModelConfig(), C.create_string_buffer(64)
+        _check(lib().b200p_model_describe(handle, name, 64, C.byref(mc)), "model_describe")
+        self.architecture = name.value.decode()
+        self.cfg = {n: getattr(mc, n) for n, _ in ModelConfig._fields_}
+        self.weights = C.cast(lib().b200p_model_weights_of(handle), C.POINTER(ModelWeights)).contents     # Llama-style models
 
     def close(self):
-        if getattr(self, "_h", None):
+        if getattr(self, "_h", None) and lib is not None:
             lib().b200p_model_free(self._h)
             self._h = None
 
@@ -585,18 +624,26 @@ class Session:
     cfg: dict with the ModelConfig fields.  The session keeps the tensors alive."""
 
     @classmethod
-    def from_model(cls, model: "Model", max_seq: int, batch: int):
-        """Session over a Model loaded from disk (Session(model_dir, max_seq) of the reference)."""
-        import torch
+    def from_model(cls, model: "Model", max_seq: int, batch: int, dtype: int = -1):
+        """Session over a loaded Model of any architecture (Session(model_dir, max_seq) of the reference).  dtype: compute
+        type, -1 for the model's own, F32 where the decoder has it."""
         self = cls.__new__(cls)
         self._weights = model                       # keeps the device memory alive
         self.cfg, self.batch, self.max_seq = dict(model.cfg), batch, max_seq
         st = _i(0)
-        self._h = lib().b200p_session_create(C.byref(model.weights), max_seq, batch, C.byref(st))
+        self._h = lib().b200p_session_open(model._h, dtype, max_seq, batch, C.byref(st))
         if not self._h:
-            raise B200PError(st.value, "session_create")
-        self._device = torch.device("cuda", torch.cuda.current_device())
+            raise B200PError(st.value, "session_open")
+        self._device = None
         return self
+
+    def _stream(self):
+        """torch's current stream, or the default stream in a process that does not use torch."""
+        import sys
+        torch = sys.modules.get("torch")
+        if torch is None or not torch.cuda.is_initialized():
+            return None
+        return torch.cuda.current_stream(self._device).cuda_stream
 
     def __init__(self, cfg: dict, weights: dict, max_seq: int, batch: int):
         self._weights = weights
@@ -634,31 +681,43 @@ class Session:
         """input_ids [batch, T] (host ints) -> (tokens [batch, max_new_tokens] numpy int32,
         (ttft_ms, decode_ms))."""
         import numpy as np
-        import torch
         a = self._ids(input_ids).reshape(self.batch, -1)
         out = np.zeros((self.batch, max_new_tokens), np.int32)
         tm = (C.c_float * 2)()
         _check(lib().b200p_session_generate(self._h, a.ctypes.data, a.shape[1], max_new_tokens, out.ctypes.data, tm,
-                                            torch.cuda.current_stream(self._device).cuda_stream), "session_generate")
+                                            self._stream()), "session_generate")
         return out, (tm[0], tm[1])
 
     def prefill_logits(self, input_ids):
         import numpy as np
-        import torch
         a = self._ids(input_ids).reshape(self.batch, -1)
         out = np.zeros((self.batch, self.cfg["vocab_size"]), np.float32)
         _check(lib().b200p_session_prefill_logits(self._h, a.ctypes.data, a.shape[1], out.ctypes.data,
-                                                  torch.cuda.current_stream(self._device).cuda_stream), "session_prefill_logits")
+                                                  self._stream()), "session_prefill_logits")
         return out
 
     def step_logits(self, token_ids):
         import numpy as np
-        import torch
         a = self._ids(token_ids).reshape(self.batch)
         out = np.zeros((self.batch, self.cfg["vocab_size"]), np.float32)
         _check(lib().b200p_session_step_logits(self._h, a.ctypes.data, out.ctypes.data,
-                                               torch.cuda.current_stream(self._device).cuda_stream), "session_step_logits")
+                                               self._stream()), "session_step_logits")
         return out
+
+    def extend(self, token_ids, want=()):
+        """The next tokens of every sequence on top of the cache (a prompt, a portion of one, or one token):
+        token_ids [batch, T]; want: indexes among the T tokens -> fp32 logits [batch, len(want), vocab]."""
+        import numpy as np
+        a = self._ids(token_ids).reshape(self.batch, -1)
+        w = self._ids(list(want))
+        out = np.zeros((self.batch, len(w), self.cfg["vocab_size"]), np.float32)
+        _check(lib().b200p_session_extend(self._h, a.ctypes.data, a.shape[1], w.ctypes.data, len(w), out.ctypes.data,
+                                          self._stream()), "session_extend")
+        return out
+
+    def reset(self):
+        """Gives the cache back: the next extend() starts new sequences."""
+        lib().b200p_session_reset(self._h)
 
     @property
     def kv_len(self) -> int:

@@ -13,6 +13,7 @@
 //   EPI_ACC32    C fp32 += A.W^T                       (O and down projections + add_f32_kernel)
 //   EPI_SILU16   W = [gate; up] (2N rows); C 16-bit = SiLU(A.gate^T) * (A.up^T)
 //                                                      (gate/up GEMMs + silu_mul_f32_kernel)
+//   EPI_GELU16   the same with the tanh form of GELU
 //
 // Both operands are K-major, so a tile is the Q.K^T case of the attention kernel:
 // TMA loads [rows][64 x 16-bit] boxes with the 128-byte swizzle into a ring of
@@ -58,6 +59,13 @@ template <int BN> struct GemmShape {
     static constexpr int SMEM_BYTES = OFF_BAR + 256;
 };
 
+// Activation of the gated epilogues on the SFU: one ex2 and one approximate divide per element.  tanh form of GELU:
+// 0.5 z (1 + tanh u) = z / (1 + e^(-2u)), u = sqrt(2/pi) (z + 0.044715 z^3).
+template <int EPI> __device__ __forceinline__ float gemm_act(float z) {
+    const float e = EPI == GEMM_EPI_GELU16 ? 1.5957691216057308f * (z + 0.044715f * z * z * z) : z;
+    return __fdividef(z, 1.f + __expf(-e));
+}
+
 struct GemmParams {
     void* C;
     long long ldc;
@@ -77,7 +85,7 @@ gemm_tc_kernel(const GemmParams p, const __grid_constant__ CUtensorMap mapA, con
                const __grid_constant__ CUtensorMap mapC) {
     using Sh = GemmShape<BN>;
     constexpr int ST = Sh::STAGES;
-    constexpr int OUT_N = EPI == GEMM_EPI_SILU16 ? BN / 2 : BN;     // output columns per tile
+    constexpr int OUT_N = gemm_gated(EPI) ? BN / 2 : BN;     // output columns per tile
     extern __shared__ __align__(1024) unsigned char smem[];
     uint64_t* bars = reinterpret_cast<uint64_t*>(smem + Sh::OFF_BAR);
     uint64_t* full = bars;                  // [ST]
@@ -115,7 +123,7 @@ gemm_tc_kernel(const GemmParams p, const __grid_constant__ CUtensorMap mapA, con
                     unsigned char* sa = smem + r.stage * Sh::STAGE_BYTES;
                     dme::mbar_arrive_expect_tx(&full[r.stage], Sh::STAGE_BYTES);
                     dme::copy_tile_2d(sa, &mapA, kb * kTK, tm * kTM, &full[r.stage]);
-                    if (EPI == GEMM_EPI_SILU16) {           // gate rows, then the matching up rows N further down
+                    if (gemm_gated(EPI)) {           // gate rows, then the matching up rows N further down
                         dme::copy_tile_2d(sa + Sh::A_BYTES, &mapW, kb * kTK, tn * OUT_N, &full[r.stage]);
                         dme::copy_tile_2d(sa + Sh::A_BYTES + Sh::B_BYTES / 2, &mapW, kb * kTK, p.N + tn * OUT_N, &full[r.stage]);
                     } else if (BN == 256) {                 // a box holds at most 256 rows; two boxes of 128 keep one map for both tile widths
@@ -157,7 +165,7 @@ gemm_tc_kernel(const GemmParams p, const __grid_constant__ CUtensorMap mapA, con
         }
     } else {
         // ---------------------------------- epilogue warps --------------------------------
-        constexpr bool OUT16 = EPI == GEMM_EPI_STORE16 || EPI == GEMM_EPI_SILU16;
+        constexpr bool OUT16 = EPI == GEMM_EPI_STORE16 || gemm_gated(EPI);
         constexpr int GCOLS = OUT16 ? 64 : 32;                // output columns per 128-byte group
         const int q = warp & 3;                               // TMEM lane quarter this warp may touch
         const int r = q * 32 + lane;                          // row inside the tile
@@ -182,16 +190,15 @@ gemm_tc_kernel(const GemmParams p, const __grid_constant__ CUtensorMap mapA, con
                 uint32_t v[GCOLS], w[32];                      // accumulator columns of this group; 128 bytes of output
                 #pragma unroll
                 for (int h = 0; h < GCOLS / 32; ++h) tc::ld_32x32b_x32(tacc + c * GCOLS + h * 32, *reinterpret_cast<uint32_t(*)[32]>(&v[h * 32]));
-                if (EPI == GEMM_EPI_SILU16) {
+                if (gemm_gated(EPI)) {
                     uint32_t u[GCOLS];
                     #pragma unroll
                     for (int h = 0; h < GCOLS / 32; ++h) tc::ld_32x32b_x32(tacc + OUT_N + c * GCOLS + h * 32, *reinterpret_cast<uint32_t(*)[32]>(&u[h * 32]));
                     tc::wait_ld();
                     #pragma unroll
-                    for (int i = 0; i < 32; ++i) {              // SiLU on the SFU: one ex2 and one approximate divide per element
+                    for (int i = 0; i < 32; ++i) {
                         const float g0 = __uint_as_float(v[2 * i]), g1 = __uint_as_float(v[2 * i + 1]);
-                        w[i] = pack2<T>(__fdividef(g0, 1.f + __expf(-g0)) * __uint_as_float(u[2 * i]),
-                                        __fdividef(g1, 1.f + __expf(-g1)) * __uint_as_float(u[2 * i + 1]));
+                        w[i] = pack2<T>(gemm_act<EPI>(g0) * __uint_as_float(u[2 * i]), gemm_act<EPI>(g1) * __uint_as_float(u[2 * i + 1]));
                     }
                 } else {
                     tc::wait_ld();
@@ -230,17 +237,17 @@ template <typename T, int BN, int EPI>
 int launch_gemm(const void* A, const void* W, void* C, int M, int N, int K, long long lda, long long ldw, long long ldc,
                 int dtype, cudaStream_t st) {
     using Sh = GemmShape<BN>;
-    constexpr int OUT_N = EPI == GEMM_EPI_SILU16 ? BN / 2 : BN;
+    constexpr int OUT_N = gemm_gated(EPI) ? BN / 2 : BN;
     const CUtensorMapDataType dt = dtype == B200P_F16 ? CU_TENSOR_MAP_DATA_TYPE_FLOAT16 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
     CUtensorMap ma, mw;
     const uint64_t ad[2] = {uint64_t(K), uint64_t(M)}, as[1] = {uint64_t(lda) * 2};
-    const uint64_t wrows = EPI == GEMM_EPI_SILU16 ? uint64_t(2) * N : uint64_t(N);
+    const uint64_t wrows = gemm_gated(EPI) ? uint64_t(2) * N : uint64_t(N);
     const uint64_t wd[2] = {uint64_t(K), wrows}, ws[1] = {uint64_t(ldw) * 2};
     const uint32_t boxa[2] = {kTK, kTM}, boxw[2] = {kTK, 128};
     cudaError_t e = make_tensor_map(&ma, dt, 2, A, ad, as, boxa, Swizzle::B128);
     if (e == cudaSuccess) e = make_tensor_map(&mw, dt, 2, W, wd, ws, boxw, Swizzle::B128);
     // C: boxes of 128 rows x 128 bytes, written (or add-reduced) from the epilogue's staging tiles
-    constexpr bool OUT16 = EPI == GEMM_EPI_STORE16 || EPI == GEMM_EPI_SILU16;
+    constexpr bool OUT16 = EPI == GEMM_EPI_STORE16 || gemm_gated(EPI);
     CUtensorMap mc;
     const uint64_t cd[2] = {uint64_t(N), uint64_t(M)}, cs[1] = {uint64_t(ldc) * (OUT16 ? 2 : 4)};
     const uint32_t boxc[2] = {OUT16 ? 64u : 32u, kTM};
@@ -271,7 +278,7 @@ int launch_gemm(const void* A, const void* W, void* C, int M, int N, int K, long
 template <typename T, int EPI>
 int launch_gemm_bn(const void* A, const void* W, void* C, int M, int N, int K, long long lda, long long ldw, long long ldc,
                    int dtype, cudaStream_t st) {
-    if (EPI == GEMM_EPI_SILU16) return launch_gemm<T, 256, EPI>(A, W, C, M, N, K, lda, ldw, ldc, dtype, st);
+    if (gemm_gated(EPI)) return launch_gemm<T, 256, EPI>(A, W, C, M, N, K, lda, ldw, ldc, dtype, st);
     // A 128 x 256 tile moves 1.5 bytes of shared memory per flop-unit against 2 for a 128 x 128 tile (both the TMA
     // writes and the MMA reads share the 128 bytes per clock of an SM), so per column it costs 3/4 of the narrow
     // tile's time; but the launch takes whole waves of tiles over the SMs.  Pick the width with the smaller
@@ -291,6 +298,7 @@ int launch_gemm_epi(int epi, const void* A, const void* W, void* C, int M, int N
         case GEMM_EPI_STORE16: return launch_gemm_bn<T, GEMM_EPI_STORE16>(A, W, C, M, N, K, lda, ldw, ldc, dtype, st);
         case GEMM_EPI_ACC32:   return launch_gemm_bn<T, GEMM_EPI_ACC32>(A, W, C, M, N, K, lda, ldw, ldc, dtype, st);
         case GEMM_EPI_STORE32: return launch_gemm_bn<T, GEMM_EPI_STORE32>(A, W, C, M, N, K, lda, ldw, ldc, dtype, st);
+        case GEMM_EPI_GELU16:  return launch_gemm_bn<T, GEMM_EPI_GELU16>(A, W, C, M, N, K, lda, ldw, ldc, dtype, st);
         case GEMM_EPI_SILU16:  return launch_gemm_bn<T, GEMM_EPI_SILU16>(A, W, C, M, N, K, lda, ldw, ldc, dtype, st);
     }
     return B200P_E_OP;
@@ -306,7 +314,7 @@ int gemm_tc(int dtype, int epi, const void* A, const void* W, void* C, int M, in
     // TMA: 16-byte aligned bases and row strides for A, W and C
     if (K % 8 != 0 || lda % 8 != 0 || ldw % 8 != 0 || lda < K || ldw < K || ldc < N) return B200P_E_RANGE;
     if (!aligned(A, 16) || !aligned(W, 16) || !aligned(C, 16)) return B200P_E_ALIGN;
-    const bool c16 = epi == GEMM_EPI_STORE16 || epi == GEMM_EPI_SILU16;
+    const bool c16 = epi == GEMM_EPI_STORE16 || gemm_gated(epi);
     if ((ldc * (c16 ? 2 : 4)) % 16 != 0) return B200P_E_ALIGN;
     if (sm_count() <= 0) return B200P_E_NO_DEVICE;
     return dtype == B200P_F16 ? launch_gemm_epi<__half>(epi, A, W, C, M, N, K, lda, ldw, ldc, dtype, st)

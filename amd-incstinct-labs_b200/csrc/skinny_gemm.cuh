@@ -55,9 +55,24 @@
 
 namespace b200p {
 
-enum SkinnyPrologue { PRO_PLAIN = 0, PRO_RMSNORM = 1 };
+enum SkinnyPrologue { PRO_PLAIN = 0, PRO_RMSNORM = 1,
+                      PRO_POSTADD = 2 };         // X = x + RMSNorm(y) * w in fp32, kept for the next reader and rounded to 16 bits (y null: X = x)
 enum SkinnyEpilogue { EPI_STORE16 = 0, EPI_ACC32 = 1, EPI_STORE32 = 2, EPI_SILU16 = 3, EPI_ROPE = 4,
-                      EPI_STORE32_BEST = 5 };   // fp32 store + running argmax key per row (decode_mega.cuh only)
+                      EPI_STORE32_BEST = 5,      // fp32 store + running argmax key per row (decode_mega.cuh only)
+                      EPI_GELU16 = 6,            // like EPI_SILU16 with the tanh form of GELU
+                      EPI_PAIRROT = 7 };         // queries whose heads are [plain | rotated] parts (SkinnyPairRot)
+// Gated epilogues: W is [2N][K], gate rows then up rows; out = act(gate) * up.
+constexpr bool epi_gated(int epi) { return epi == EPI_SILU16 || epi == EPI_GELU16; }
+// A group's rows g and g + 8 meet in one thread.
+constexpr bool epi_paired(int epi) { return epi_gated(epi) || epi == EPI_ROPE || epi == EPI_PAIRROT; }
+
+// 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))
+__device__ __forceinline__ float gelu_tanh(float z) {
+    return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+template <int EPI> __device__ __forceinline__ float gate_act(float g) {
+    return EPI == EPI_GELU16 ? gelu_tanh(g) : g / (1.f + expf(-g));
+}
 
 // EPI_ROPE: W is the concatenated Q/K/V projection; the epilogue is the reference's bias add,
 // rotate-half RoPE and KV-cache scatter (forward.hpp:135-148, 211-224; rocblas_gemm.hpp:56-63)
@@ -73,6 +88,18 @@ struct SkinnyRope {
     int pos0, nQH, nKVH, D, max_seq;
 };
 
+// EPI_PAIRROT: W is a query projection whose heads are `plain` rows without and `rotated` rows with rotary positions
+// (multiples of 16).  Rotated rows come in groups of 16, the first members of eight pairs, then the second members,
+// so each pair meets in one thread whatever the checkpoint's pairing was.  Plain columns go to `out` [M][heads * plain]
+// (ldo), rotated ones to columns rot_col.. of rot_out [M * heads][rot_ld].  Row m of X is token m % Tn of its sequence.
+struct SkinnyPairRot {
+    const float* cos_t;     // [max_seq][rotated / 2]
+    const float* sin_t;
+    const int* pos_dev;     // position of a sequence's first token, read on the device (null: pos0)
+    void* rot_out;
+    int pos0, Tn, plain, rotated, heads, rot_ld, rot_col, max_seq;
+};
+
 struct SkinnyArgs {
     const void*  W;        // [N][K] 16-bit (EPI_SILU16: [2N][K], gate rows then up rows)
     const void*  X16;      // PRO_PLAIN:   [M][ldx] 16-bit activations
@@ -83,7 +110,12 @@ struct SkinnyArgs {
     void*        out;      // [M][ldo] 16-bit or fp32
     int M, N, K, ldx, ldo;
     float eps;
+    int norm_n;            // columns the norm's mean is over (0: K; columns past them are zero padding)
+    int ldx32;             // row stride of X32 (0: K)
+    const float* Y32;      // PRO_POSTADD: [M][K] fp32 sublayer output, or null
+    float* x_out;          // PRO_POSTADD with Y32: [M][K] fp32, the sum (another buffer than X32)
     SkinnyRope rope;       // EPI_ROPE only
+    SkinnyPairRot pair;    // EPI_PAIRROT only
     int* abort_word;       // streaming kernel: the abort word its bounded waits poll and raise.  A caller that
                            // launches many of these on one stream (the runtime's decode step) owns one word,
                            // clears it before the step and reads it after; null: a per-launch slot is taken.
@@ -110,14 +142,14 @@ __device__ __forceinline__ void skinny_prologue(const SkinnyArgs& a, T* xs, floa
         for (int m = warp; m < Mp; m += kSkinnyWarps) {
             T* dst = xs + size_t(m) * xstride;
             if (m < a.M) {
-                const float* x = a.X32 + size_t(m) * K;
+                const float* x = a.X32 + size_t(m) * (a.ldx32 ? a.ldx32 : K);
                 float ss = 0.f;
                 for (int q = lane; q < K / 4; q += 32) {
                     const float4 v = *reinterpret_cast<const float4*>(x + 4 * q);
                     ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
                 }
                 ss = wave::dpp::reduce_sum(ss);
-                const float inv = rsqrtf(ss / K + a.eps);
+                const float inv = rsqrtf(ss / (a.norm_n ? a.norm_n : K) + a.eps);
                 for (int q = lane; q < K / 4; q += 32) {
                     const float4 v = *reinterpret_cast<const float4*>(x + 4 * q);
                     const uint2 wv = *reinterpret_cast<const uint2*>(nw + 4 * q);
@@ -139,7 +171,7 @@ __device__ __forceinline__ void skinny_prologue(const SkinnyArgs& a, T* xs, floa
         const int m = warp / wpr, part = warp % wpr;
         const int quads = K / 4, qper = (quads + wpr - 1) / wpr;
         const int q0 = part * qper, q1 = min(q0 + qper, quads);
-        const float* x = a.X32 + size_t(m) * K;
+        const float* x = a.X32 + size_t(m) * (a.ldx32 ? a.ldx32 : K);
         const T* xe = EMB && m < a.M ? static_cast<const T*>(a.Xemb) + size_t(a.Xids[m]) * K : nullptr;
         auto ldx = [&](int q) -> float4 {                       // four elements of row m as fp32
             if (!EMB) return *reinterpret_cast<const float4*>(x + 4 * q);
@@ -168,7 +200,7 @@ __device__ __forceinline__ void skinny_prologue(const SkinnyArgs& a, T* xs, floa
                 ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
             }
         }
-        const float inv_k = 1.f / float(K);                     // off the chain: computed while the loads are in flight
+        const float inv_k = 1.f / float(a.norm_n ? a.norm_n : K);                     // off the chain: computed while the loads are in flight
         ss = wave::dpp::reduce_sum(ss);
         if (lane == 0) part_ss[warp] = ss;
         skinny_barrier();
@@ -201,6 +233,72 @@ __device__ __forceinline__ void skinny_prologue(const SkinnyArgs& a, T* xs, floa
                 put(q, ldx(q), ldw(q));
         } else {
             for (int q = q0 + lane; q < q1; q += 32) *reinterpret_cast<uint2*>(dst + 4 * q) = make_uint2(0u, 0u);
+        }
+    } else if (PRO == PRO_POSTADD) {
+        // 8 / Mp warps share a row (one each from eight rows on, then rows warp and warp + 8); x and y of up to CACHE
+        // quads per lane are in registers before the sum of squares is known
+        constexpr int CACHE = 4;
+        const int wpr = Mp >= kSkinnyWarps ? 1 : kSkinnyWarps / Mp;
+        const int part = warp % wpr;
+        const int quads = K / 4, qper = (quads + wpr - 1) / wpr;
+        const int q0 = part * qper, q1 = min(q0 + qper, quads);
+        const T* nw = static_cast<const T*>(a.norm_w);
+        const float inv_n = 1.f / float(a.norm_n ? a.norm_n : K);
+        for (int m = warp / wpr; m < Mp; m += kSkinnyWarps / wpr) {          // one trip unless Mp = 16
+            T* dst = xs + size_t(m) * xstride;
+            const bool live = m < a.M;
+            const float* x = a.X32 + size_t(live ? m : 0) * K;
+            const float* y = a.Y32 ? a.Y32 + size_t(live ? m : 0) * K : nullptr;
+            float4 cx[CACHE], cy[CACHE];
+            float ss = 0.f;
+            #pragma unroll
+            for (int it = 0; it < CACHE; ++it) {
+                const int q = q0 + lane + 32 * it;
+                cx[it] = cy[it] = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (live && q < q1) {
+                    cx[it] = *reinterpret_cast<const float4*>(x + 4 * q);
+                    if (y) cy[it] = *reinterpret_cast<const float4*>(y + 4 * q);
+                }
+                ss += cy[it].x * cy[it].x + cy[it].y * cy[it].y + cy[it].z * cy[it].z + cy[it].w * cy[it].w;
+            }
+            if (live && y)
+                for (int q = q0 + lane + 32 * CACHE; q < q1; q += 32) {
+                    const float4 v = *reinterpret_cast<const float4*>(y + 4 * q);
+                    ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+                }
+            ss = wave::dpp::reduce_sum(ss);
+            if (wpr > 1) {
+                if (lane == 0) part_ss[warp] = ss;
+                skinny_barrier();
+                ss = 0.f;
+                #pragma unroll
+                for (int w = 0; w < kSkinnyWarps; ++w) ss += (w >= (warp / wpr) * wpr && w < (warp / wpr + 1) * wpr) ? part_ss[w] : 0.f;
+            }
+            const float inv = rsqrtf(ss * inv_n + a.eps);
+            auto put = [&](int q, const float4& xv, const float4& yv) {
+                float4 o = xv;
+                if (y) {
+                    const uint2 wv = *reinterpret_cast<const uint2*>(nw + 4 * q);
+                    const T* w4 = reinterpret_cast<const T*>(&wv);
+                    o.x += yv.x * inv * to_float(w4[0]); o.y += yv.y * inv * to_float(w4[1]);
+                    o.z += yv.z * inv * to_float(w4[2]); o.w += yv.w * inv * to_float(w4[3]);
+                    if (live && blockIdx.x == 0) *reinterpret_cast<float4*>(a.x_out + size_t(m) * K + 4 * q) = o;
+                }
+                *reinterpret_cast<uint2*>(dst + 4 * q) = make_uint2(pack2<T>(o.x, o.y), pack2<T>(o.z, o.w));
+            };
+            #pragma unroll
+            for (int it = 0; it < CACHE; ++it) {
+                const int q = q0 + lane + 32 * it;
+                if (q < q1) put(q, cx[it], cy[it]);
+            }
+            for (int q = q0 + lane + 32 * CACHE; q < q1; q += 32) {
+                float4 xv = make_float4(0.f, 0.f, 0.f, 0.f), yv = xv;
+                if (live) {
+                    xv = *reinterpret_cast<const float4*>(x + 4 * q);
+                    if (y) yv = *reinterpret_cast<const float4*>(y + 4 * q);
+                }
+                put(q, xv, yv);
+            }
         }
     } else {
         // 16-byte vectors, two rows at a time and up to three vectors per row and thread: the loads of a batch are all
@@ -276,13 +374,19 @@ __device__ __forceinline__ void skinny_epilogue_fetch(const SkinnyArgs& a, int g
     }
 }
 
+// Position and table offset of pair j of row m (EPI_PAIRROT).
+__device__ __forceinline__ size_t pair_angle(const SkinnyPairRot& r, int m, int j) {
+    const int pos = min((r.pos_dev ? *r.pos_dev : r.pos0) + m % r.Tn, r.max_seq - 1);
+    return size_t(pos) * (r.rotated / 2) + j;
+}
+
 // red[warp][lane][4 * mh + c]: the m16n8 C fragment of the MMA over rows 8 mh .. 8 mh + 7 of X.
 template <typename T, int EPI, int R, int MH>
 __device__ __forceinline__ void skinny_epilogue(const SkinnyArgs& a, const float (*red)[32][4 * MH], int grp, int tid, bool use_prev, float prev,
                                                 unsigned long long* best = nullptr, const EpiAhead<MH>* ahead = nullptr) {
     #pragma unroll
     for (int mh = 0; mh < MH; ++mh) {
-        if (EPI == EPI_SILU16) {
+        if (epi_gated(EPI)) {
             if (tid < 64) {
                 const int l = tid % 32, sel = tid / 32;
                 float gate = 0.f, up = 0.f;
@@ -290,7 +394,7 @@ __device__ __forceinline__ void skinny_epilogue(const SkinnyArgs& a, const float
                 for (int w = 0; w < kSkinnyWarps; ++w) { gate += red[w][l][4 * mh + sel]; up += red[w][l][4 * mh + 2 + sel]; }
                 const int m = 8 * mh + 2 * (l % 4) + sel, p = grp * 8 + l / 4;
                 if (m < a.M && p < a.N)
-                    static_cast<T*>(a.out)[size_t(m) * a.ldo + p] = from_float<T>((gate / (1.f + expf(-gate))) * up);
+                    static_cast<T*>(a.out)[size_t(m) * a.ldo + p] = from_float<T>(gate_act<EPI>(gate) * up);
             }
         } else if (EPI == EPI_ROPE) {
             if (tid < 64) {
@@ -324,6 +428,27 @@ __device__ __forceinline__ void skinny_epilogue(const SkinnyArgs& a, const float
                         const int kvh = is_k ? slot - r.nQH : slot - r.nQH - r.nKVH;
                         T* dst = static_cast<T*>(is_k ? r.kcache : r.vcache) + ((size_t(m) * r.nKVH + kvh) * r.max_seq + pos) * r.D;
                         dst[d] = o0; dst[d + half] = o1;
+                    }
+                }
+            }
+        } else if (EPI == EPI_PAIRROT) {
+            if (tid < 64) {
+                const SkinnyPairRot& r = a.pair;
+                const int l = tid % 32, sel = tid / 32;
+                float x0 = 0.f, x1 = 0.f;
+                #pragma unroll
+                for (int w = 0; w < kSkinnyWarps; ++w) { x0 += red[w][l][4 * mh + sel]; x1 += red[w][l][4 * mh + 2 + sel]; }
+                const int m = 8 * mh + 2 * (l % 4) + sel;
+                const int per_head = r.plain + r.rotated, head = grp * 16 / per_head, j = grp * 16 % per_head;
+                if (m < a.M && head < r.heads) {
+                    if (j < r.plain) {
+                        T* row = static_cast<T*>(a.out) + size_t(m) * a.ldo + size_t(head) * r.plain + j + l / 4;
+                        row[0] = from_float<T>(x0); row[8] = from_float<T>(x1);
+                    } else {
+                        const size_t t = pair_angle(r, m, (j - r.plain) / 2 + l / 4);
+                        const float c = r.cos_t[t], sn = r.sin_t[t];
+                        T* row = static_cast<T*>(r.rot_out) + (size_t(m) * r.heads + head) * r.rot_ld + r.rot_col + (j - r.plain) + l / 4;
+                        row[0] = from_float<T>(x0 * c - x1 * sn); row[8] = from_float<T>(x1 * c + x0 * sn);
                     }
                 }
             }
@@ -366,7 +491,7 @@ skinny_gemm_kernel(const SkinnyArgs a) {
     __shared__ float red[2][kSkinnyWarps][32][4 * MH];          // double-buffered by group
     __shared__ __align__(16) float part_ss[kSkinnyWarps];
     constexpr int DEPTH = 8 / R;
-    static_assert(R == 2 || (EPI != EPI_SILU16 && EPI != EPI_ROPE), "paired epilogues need both halves");
+    static_assert(R == 2 || !epi_paired(EPI), "paired epilogues need both halves");
     const int warp = threadIdx.x / 32, lane = threadIdx.x % 32;
     const int g = lane / 4, t4 = lane % 4;
     const int K = a.K, xstride = K + kSkinnyXPad;
@@ -374,10 +499,10 @@ skinny_gemm_kernel(const SkinnyArgs a) {
 
     // Row groups: group `grp` is 8 * R rows of W (8 row pairs for the paired epilogues); the CTA
     // takes groups blockIdx.x, blockIdx.x + gridDim.x, ...
-    const int ngroups = (EPI == EPI_SILU16) ? (a.N + 7) / 8 : (a.N + 8 * R - 1) / (8 * R);
+    const int ngroups = (epi_gated(EPI)) ? (a.N + 7) / 8 : (a.N + 8 * R - 1) / (8 * R);
     auto row_ptrs = [&](int grp, const char*& wA, const char*& wB) {
         size_t rowA, rowB;
-        if (EPI == EPI_SILU16) {
+        if (epi_gated(EPI)) {
             const int p = min(grp * 8 + g, a.N - 1);            // pair index: gate row p, up row N + p
             rowA = size_t(p); rowB = size_t(a.N) + size_t(p);
         } else if (EPI == EPI_ROPE) {
@@ -518,7 +643,7 @@ skinny_stream_kernel(const SkinnyArgs a, int nstages, int slab_cols, int* status
     const int x_bytes = ((Mp * xstride * 2 + 127) / 128) * 128;
     T* xs = reinterpret_cast<T*>(skinny_smem);
     unsigned char* stages = skinny_smem + x_bytes;
-    const int ngroups = (EPI == EPI_SILU16) ? (a.N + 7) / 8 : (a.N + 15) / 16;
+    const int ngroups = (epi_gated(EPI)) ? (a.N + 7) / 8 : (a.N + 15) / 16;
 
     if (threadIdx.x == 0) {
         for (int s = 0; s < nstages; ++s) { dme::mbar_init(&full_bar[s], 1); dme::mbar_init(&empty_bar[s], kSkinnyWarps); }
@@ -540,7 +665,7 @@ skinny_stream_kernel(const SkinnyArgs a, int nstages, int slab_cols, int* status
                     dme::mbar_arrive_expect_tx(&full_bar[stage], uint32_t(16 * cols * 2));
                     for (int r = 0; r < 16; ++r) {
                         size_t row;
-                        if (EPI == EPI_SILU16)    row = r < 8 ? size_t(min(grp * 8 + r, a.N - 1)) : size_t(a.N) + size_t(min(grp * 8 + r - 8, a.N - 1));
+                        if (epi_gated(EPI))    row = r < 8 ? size_t(min(grp * 8 + r, a.N - 1)) : size_t(a.N) + size_t(min(grp * 8 + r - 8, a.N - 1));
                         else if (EPI == EPI_ROPE) { const int cph = a.rope.D / 16;
                                                     row = size_t(grp / cph) * a.rope.D + size_t(grp % cph) * 8 + (r & 7) + (r >= 8 ? a.rope.D / 2 : 0); }
                         else                      row = size_t(min(grp * 16 + r, a.N - 1));
@@ -678,14 +803,16 @@ template <typename T, int PRO, int EPI, int MH>
 int launch_skinny_mh(const SkinnyArgs& a, cudaStream_t st) {
     if (a.M < 1 || a.M > kSkinnyMaxM || a.K < 16 || a.K % 16 != 0 || a.N < 1) return B200P_E_RANGE;
     if (PRO == PRO_PLAIN && (a.ldx % 8 != 0 || !aligned(a.X16, 16))) return B200P_E_RANGE;
-    if (PRO == PRO_RMSNORM && (!aligned(a.X32, 16) || !aligned(a.norm_w, 8))) return B200P_E_RANGE;
+    if (PRO == PRO_RMSNORM && (!aligned(a.X32, 16) || !aligned(a.norm_w, 8) || a.ldx32 % 4 != 0)) return B200P_E_RANGE;
+    if (PRO == PRO_POSTADD && (!aligned(a.X32, 16) || !aligned(a.Y32, 16) || !aligned(a.x_out, 16) || !aligned(a.norm_w, 8))) return B200P_E_RANGE;
+    if (EPI == EPI_PAIRROT && (a.pair.plain % 16 != 0 || a.pair.rotated % 16 != 0 || a.N != a.pair.heads * (a.pair.plain + a.pair.rotated))) return B200P_E_RANGE;
     if (!aligned(a.W, 16)) return B200P_E_RANGE;               // bulk copies need 16 bytes; the register kernel's 32-byte loads are checked below
     const int Mp = a.M <= 1 ? 1 : a.M <= 2 ? 2 : a.M <= 4 ? 4 : a.M <= 8 ? 8 : 16;
     const size_t smem = size_t(Mp) * (a.K + kSkinnyXPad) * 2;
     if (smem > 190 * 1024) return B200P_E_RANGE;
     if (EPI == EPI_ROPE && (a.rope.D % 16 != 0 || a.N != (a.rope.nQH + 2 * a.rope.nKVH) * a.rope.D)) return B200P_E_RANGE;
     const int sms = sm_count() > 0 ? sm_count() : 148;
-    constexpr bool paired = EPI == EPI_SILU16 || EPI == EPI_ROPE;
+    constexpr bool paired = epi_paired(EPI);
     const bool pdl = tuning(KNOB_RUNTIME_PDL, 1) != 0;
     if (tuning(KNOB_RUNTIME_SKINNY, 2) == 2 && aligned(a.W, 16)) {
         // W staged through shared memory by a producer thread (skinny_stream_kernel), one CTA per SM
@@ -698,7 +825,7 @@ int launch_skinny_mh(const SkinnyArgs& a, cudaStream_t st) {
         // A few more row groups than SMs (the decode step's Q/K/V: 160 on 148), each one stage long: with one CTA per
         // SM a dozen CTAs would take two groups one after the other and the whole grid would wait for them.  One CTA
         // per group with a single stage instead: two of them fit an SM and run side by side.
-        const int groups_all = EPI == EPI_SILU16 ? (a.N + 7) / 8 : (a.N + 15) / 16;
+        const int groups_all = epi_gated(EPI) ? (a.N + 7) / 8 : (a.N + 15) / 16;
         // (the two-fragment kernel holds too many registers for two CTAs of 288 threads on an SM)
         const bool one_group_ctas = MH == 1 && groups_all > sms && groups_all <= 2 * sms && a.K <= slab_cols &&
                                     x_bytes + stage_bytes + 8704 * MH + 1024 <= 113 * 1024 && nstages >= 2;
@@ -730,7 +857,7 @@ int launch_skinny_mh(const SkinnyArgs& a, cudaStream_t st) {
     if (!aligned(a.W, 32)) return B200P_E_RANGE;               // the register kernel loads 32-byte vectors of W
     // 8-row groups when 16-row groups would leave a third of the CTA slots (2 per SM) empty
     const bool half_rows = !paired && (a.N + 15) / 16 < (4 * sms) / 3;
-    const int ngroups = EPI == EPI_SILU16 ? (a.N + 7) / 8 : half_rows ? (a.N + 7) / 8 : (a.N + 15) / 16;
+    const int ngroups = epi_gated(EPI) ? (a.N + 7) / 8 : half_rows ? (a.N + 7) / 8 : (a.N + 15) / 16;
     const int grid = ngroups < 2 * sms ? ngroups : 2 * sms;      // CTAs loop over their groups, loads running ahead
     void (*kern)(SkinnyArgs) = skinny_gemm_kernel<T, PRO, EPI, 2, MH>;
     if constexpr (!paired) { if (half_rows) kern = skinny_gemm_kernel<T, PRO, EPI, 1, MH>; }

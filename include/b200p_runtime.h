@@ -74,12 +74,26 @@ b200p_model* b200p_model_load(const char* model_dir, int* status);
 const b200p_model_weights* b200p_model_weights_of(const b200p_model* model);
 void b200p_model_free(b200p_model* model);
 
+/* Other decoders: b200p_model_load also reads a directory with config.json and model.safetensors; config.json's
+ * "architecture" picks the decoder from the library's registry (B200P_E_OP: not known).  b200p_model_create makes the
+ * same model from caller-owned device tensors (config_json: the text of config.json; shapes: the ranks' dimensions one
+ * tensor after the other); missing tensors give B200P_E_IO, wrong shapes B200P_E_DIM.
+ * b200p_model_describe: the architecture's name ("Llama" for the meta.json format) and the configuration; fields that
+ * an architecture does not have (its layers differ, say) are 0. */
+b200p_model* b200p_model_create(const char* config_json, int n_tensors, const char* const* names, const void* const* pointers,
+                                const int* dtypes, const int* ranks, const long long* shapes, int* status);
+int b200p_model_describe(const b200p_model* model, char* architecture, int cap, b200p_model_config* cfg);
+
 typedef struct b200p_session b200p_session;
 
 /* Session(model, max_seq) (session.hpp:253-259) for `batch` sequences.
  * Returns NULL and sets *status on failure. */
 b200p_session* b200p_session_create(const b200p_model_weights* weights, int max_seq, int batch, int* status);
 void b200p_session_destroy(b200p_session* s);
+/* The same for any model, whatever its architecture.  dtype: compute type, B200P_BF16 / B200P_F16 / B200P_F32, or -1 for
+ * the model's own.  B200P_E_DTYPE where the decoder has no kernels of that type (B200P_F32, true 32-bit throughout:
+ * Maposun only). */
+b200p_session* b200p_session_open(const b200p_model* model, int dtype, int max_seq, int batch, int* status);
 
 /* Session::generate (session.hpp:263-296): greedy decoding.
  * input_ids: host, [batch, T] token ids; out_tokens: host, [batch, max_new_tokens].
@@ -98,6 +112,14 @@ int b200p_session_prefill_logits(b200p_session* s, const int* input_ids, int T, 
 /* One more token per sequence on top of the current cache (teacher forcing):
  * feeds token_ids [batch] (host) at position kv_len, returns logits [batch, vocab]. */
 int b200p_session_step_logits(b200p_session* s, const int* token_ids, float* logits, b200p_stream_t stream);
+
+/* The next T tokens of every sequence on top of the current cache: a whole prompt, a portion of one, or one token.
+ * input_ids: host, [batch, T].  want: host, n_want indexes among the T tokens whose logits are asked for (may be none);
+ * logits: host, fp32 [batch, n_want, vocab].  b200p_session_reset gives the cache back: the next tokens start new
+ * sequences. */
+int b200p_session_extend(b200p_session* s, const int* input_ids, int T, const int* want, int n_want, float* logits,
+                         b200p_stream_t stream);
+void b200p_session_reset(b200p_session* s);
 
 /* The decode step's projection kernel on its own: Y[M, N] = X[M, K] . W[N, K]^T for M <= 16,
  * 16-bit operands, fp32 accumulation.  Stands in for the rocBLAS calls of the decode step
