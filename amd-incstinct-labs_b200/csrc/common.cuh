@@ -35,6 +35,7 @@ enum Knob {
     KNOB_GEMM_TILE_N,           // 128 or 256: force the tensor-core GEMM's tile width (0: chosen from the shape)
     KNOB_RUNTIME_MEGA,          // 1: the greedy loop's decode steps run as one persistent cooperative kernel, 0: kernel per phase (default)
     KNOB_RUNTIME_MEGA_AHEAD,    // persistent decode kernel: stages of L2 prefetch in front of the shared-memory ring's loads
+    KNOB_LATENT_PLAIN,          // 1: latent attention of 16-bit sessions on the plain kernel as well
     KNOB_COUNT
 };
 

@@ -49,5 +49,7 @@ struct LatentAttn {
 
 // Any shape, bf16 or fp32 (fp32 arithmetic throughout).  Expanded form.
 int latent_attn_plain(const LatentAttn& a, cudaStream_t st);
+// tcgen05 (bf16; dim and vdim up to 128, rot up to 64; B200P_E_RANGE otherwise, nothing launched).  Expanded form.
+int latent_attn_prefill(const LatentAttn& a, cudaStream_t st);
 
 } // namespace b200p
