@@ -195,6 +195,8 @@ struct LatentState {
     // activations of the current scratch
     float *proj = nullptr, *y = nullptr, *gu = nullptr;
     void *x16 = nullptr, *cq = nullptr, *q = nullptr, *attn = nullptr, *act = nullptr;
+    float *x2 = nullptr, *part_o = nullptr, *part_ml = nullptr;        // few tokens: the other residual buffer; attention's partial results
+    void* q_abs = nullptr;
     void* kv = nullptr;                                // expanded keys and values [batch][N][kv_row]
 };
 LatentState* latent(const b200p_session* s) { return static_cast<LatentState*>(s->decoder.get()); }
@@ -204,6 +206,7 @@ LatentState* latent(const b200p_session* s) { return static_cast<LatentState*>(s
 template <typename T>
 __global__ void __launch_bounds__(256)
 postnorm_add_kernel(float* __restrict__ X, const float* __restrict__ Y, const T* __restrict__ W, T* __restrict__ X16, int rows, int H, int n, float eps) {
+    griddep_launch_dependents();
     const int r = blockIdx.x * (blockDim.x / 32) + threadIdx.x / 32, lane = threadIdx.x % 32;
     if (r >= rows) return;
     float* x = X + size_t(r) * H;
@@ -365,8 +368,74 @@ int layers_gemm(b200p_session* s, int Tn, int pos0, cudaStream_t st) {
     return B200P_OK;
 }
 
+// ---- few tokens -------------------------------------------------------------------------------------------
+// Whether M tokens run on the streaming kernels and the absorbed attention.
+bool few_tokens(const b200p_session* s, int M) {
+    if (!skinny_ok(s, M) || tuning(KNOB_LATENT_PLAIN, 0) != 0) return false;
+    for (const LatentLayer& l : latent(s)->spec.layers) if (!latent_step_ok(l.mix.dims(), M)) return false;
+    return true;
+}
+
+// Nine launches a layer, each a programmatic dependent of the one before.  The norms on the sublayers' outputs and the
+// residual adds are prologues of whatever reads x next (PRO_POSTADD: every CTA forms the sum, CTA 0 keeps it in the other
+// of two buffers), so y and the norm's weights travel along as `pending`.
+int layers_few(b200p_session* s, int Tn, int pos0, cudaStream_t st, const int* pos_dev) {
+    using T = __nv_bfloat16;
+    LatentState* L = latent(s);
+    const int M = s->batch * Tn, H = L->H, n = L->spec.width;
+    float *x = s->hidden, *other = L->x2;
+    const float* pending = nullptr;
+    const void* pending_w = s->final_norm;              // any valid norm weights while nothing is pending
+    auto args = [&](const void* W, void* out, int N, int K, int ldo) {
+        SkinnyArgs a{};
+        a.M = M; a.eps = s->eps; a.abort_word = s->d_abort; a.W = W; a.out = out; a.N = N; a.K = K; a.ldo = ldo;
+        ++s->gemm_calls;
+        return a;
+    };
+    auto read_x = [&](SkinnyArgs& a) {                  // X = x + norm(pending)
+        a.X32 = x; a.Y32 = pending; a.x_out = other; a.norm_w = pending_w; a.norm_n = n;
+        if (pending) std::swap(x, other);
+        pending = nullptr;
+    };
+    for (size_t li = 0; li < L->spec.layers.size(); ++li) {
+        const LatentLayer& ly = L->spec.layers[li];
+        const LatentWeights& w = L->w[li];
+        const LatentDims d = ly.mix.dims();
+        SkinnyArgs a = args(w.proj, L->proj, d.proj_row(), H, d.proj_row());
+        read_x(a);
+        if (int e = launch_skinny<T, PRO_POSTADD, EPI_STORE32>(a, st)) return e;
+        a = args(w.uq, L->q, d.q_row(), d.qrank, d.heads * d.dim);
+        a.X32 = L->proj; a.ldx32 = d.proj_row(); a.norm_w = w.q_norm; a.norm_n = ly.mix.q_rank;
+        a.pair = SkinnyPairRot{L->rot[li].first, L->rot[li].second, pos_dev, L->q_abs, pos0, Tn, d.dim, d.rot, d.heads, d.cache_row(), d.rank, s->max_seq};
+        if (int e = launch_skinny<T, PRO_RMSNORM, EPI_PAIRROT>(a, st)) return e;
+        LatentStep p{d, s->batch, Tn, pos0, s->max_seq, pos_dev, float(ly.mix.scale), s->eps, ly.mix.kv_rank, w.sink, w.ukT,
+                     static_cast<const T*>(w.kv) + size_t(d.heads) * d.dim * d.rank, w.kv_norm, L->rot[li].first, L->rot[li].second,
+                     L->proj, L->q, L->q_abs, L->cache[li], L->part_o, L->part_ml, L->attn, s->d_attn_status};
+        if (int e = latent_step_absorb(p, st)) return e;
+        if (int e = latent_step_attend(p, st)) return e;
+        if (int e = latent_step_values(p, st)) return e;
+        a = args(w.o, L->y, H, d.v_row(), H);
+        a.X16 = L->attn; a.ldx = d.v_row();
+        if (int e = launch_skinny<T, PRO_PLAIN, EPI_STORE32>(a, st)) return e;
+        pending = L->y; pending_w = w.norm1;
+        if (!ly.ff) continue;
+        const int F = pad16(ly.ff);
+        a = args(w.gu, L->act, F, H, F);
+        read_x(a);
+        if (int e = launch_skinny<T, PRO_POSTADD, EPI_GELU16>(a, st)) return e;
+        a = args(w.down, L->y, H, F, H);
+        a.X16 = L->act; a.ldx = F;
+        if (int e = launch_skinny<T, PRO_PLAIN, EPI_STORE32>(a, st)) return e;
+        pending = L->y; pending_w = w.norm2;
+    }
+    postnorm_add_kernel<T><<<blocks(size_t(M) * 32), 256, 0, st>>>(x, pending, static_cast<const T*>(pending_w), static_cast<T*>(L->x16), M, H, n, s->eps);
+    s->final_x = x;
+    return launched();
+}
+
 template <typename T>
 int latent_run_layers(b200p_session* s, int Tn, int pos0, cudaStream_t st, const int* pos_dev) {
+    if (!std::is_same_v<T, float> && few_tokens(s, s->batch * Tn)) return layers_few(s, Tn, pos0, st, pos_dev);
     if (pos_dev) pos0 = s->kv_len;
     return layers_gemm<T>(s, Tn, pos0, st);
 }
@@ -383,11 +452,12 @@ int latent_alloc_scratch(b200p_session* s, int M) {
     if ((c = s->alloc_scratch(&L->attn, m * L->max_v * e))) return int(c);
     if ((c = s->alloc_scratch(&L->y, m * L->H * 4))) return int(c);
     if ((c = s->alloc_scratch(&L->act, m * L->max_ff * e))) return int(c);
+    if ((c = s->alloc_scratch(&L->x2, std::min<size_t>(m, kSkinnyMaxM) * L->H * 4))) return int(c);
     if ((c = s->alloc_scratch(&L->gu, m * 2 * L->max_ff * 4))) return int(c);
     return B200P_OK;
 }
 
-bool latent_graph_step(const b200p_session*) { return false; }
+bool latent_graph_step(const b200p_session* s) { return few_tokens(s, s->batch); }
 int latent_gemms_per_step(const b200p_session* s) {
     int n = 0;
     for (const LatentLayer& l : latent(s)->spec.layers) n += l.ff ? 5 : 3;
@@ -399,7 +469,7 @@ template <typename T>
 int build_weights(b200p_session* s, const b200p_model* m) {
     LatentState* L = latent(s);
     const LatentSpec& spec = L->spec;
-    const int H = L->H, D = spec.width;
+    const int H = L->H;
     int rc = B200P_OK;
     auto zeros = [&](size_t n, size_t esz) -> void* {
         void* p = nullptr;
@@ -479,7 +549,6 @@ int build_weights(b200p_session* s, const b200p_model* m) {
             w.down = padded(p + "mlp.down", H, F);
         }
     }
-    (void)D;
     return rc;
 }
 
@@ -535,6 +604,18 @@ int latent_build(b200p_session* s, const b200p_model* m) {
     s->skinny_max_k = max_k;
     s->skinny_usable = s->dtype != B200P_F32;
     if (cudaError_t e = s->alloc(&L->kv, size_t(s->batch) * s->max_seq * L->max_kv * esz)) return int(e);
+    if (s->dtype == B200P_BF16) {                         // the absorbed attention's queries and partial results
+        size_t parts = 0, part_floats = 0, abs = 0;
+        for (const LatentLayer& ly : L->spec.layers) {
+            const LatentDims d = ly.mix.dims();
+            const size_t n = latent_step_partials(d);
+            parts = std::max(parts, n); part_floats = std::max(part_floats, n * d.rank);
+            abs = std::max(abs, size_t(kSkinnyMaxM) * d.heads * d.cache_row());
+        }
+        if (cudaError_t e = s->alloc(&L->part_o, part_floats * 4)) return int(e);
+        if (cudaError_t e = s->alloc(&L->part_ml, parts * 8)) return int(e);
+        if (cudaError_t e = s->alloc(&L->q_abs, abs * 2)) return int(e);
+    }
     if (cudaError_t e = s->alloc(&s->d_attn_status, 16)) return int(e);
     return int(cudaMemset(s->d_attn_status, 0, 16));
 }

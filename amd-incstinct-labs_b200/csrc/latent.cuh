@@ -47,6 +47,31 @@ struct LatentAttn {
     void* out;                     // [batch * Tn][v_row], gated
 };
 
+// A few new tokens per sequence (M = batch * Tn <= 16) on the latent cache: absorbed form, bf16, three launches.
+struct LatentStep {
+    LatentDims d;
+    int batch, Tn, pos0, max_seq;
+    const int* pos_dev;            // position of the first new token, read on the device (null: pos0)
+    float scale, eps;
+    int kv_rank;                   // columns of the latent without padding
+    const float* sink;             // [heads] or null
+    const void *ukT, *uv;          // [heads][rank][dim], [heads * vdim][rank]
+    const void* kv_norm;           // [rank]
+    const float *cos_t, *sin_t;    // [max_seq][rot / 2]
+    const float* proj;             // [M][proj_row]
+    const void* q_plain;           // [M][heads * dim]
+    void* q_abs;                   // [M * heads][cache_row]: the rotated part is there already
+    void* cache;                   // [batch][max_seq][cache_row]
+    float *part_o, *part_ml;       // splits' partial results: latent_step_partials(d) rows of `rank` and of 2 floats
+    void* out;                     // [M][v_row], gated
+    int* abort_word;
+};
+bool latent_step_ok(const LatentDims& d, int M);
+size_t latent_step_partials(const LatentDims& d);
+int latent_step_absorb(const LatentStep& a, cudaStream_t st);     // latents and rotated keys into the cache; W_uk^T q
+int latent_step_attend(const LatentStep& a, cudaStream_t st);     // splits of the cache -> partial weighted latents
+int latent_step_values(const LatentStep& a, cudaStream_t st);     // merge, W_uv, gate
+
 // Any shape, bf16 or fp32 (fp32 arithmetic throughout).  Expanded form.
 int latent_attn_plain(const LatentAttn& a, cudaStream_t st);
 // tcgen05 (bf16; dim and vdim up to 128, rot up to 64; B200P_E_RANGE otherwise, nothing launched).  Expanded form.
