@@ -196,7 +196,7 @@ struct LatentState {
     float *proj = nullptr, *y = nullptr, *gu = nullptr;
     void *x16 = nullptr, *cq = nullptr, *q = nullptr, *attn = nullptr, *act = nullptr;
     float *x2 = nullptr, *part_o = nullptr, *part_ml = nullptr;        // few tokens: the other residual buffer; attention's partial results
-    void* q_abs = nullptr;
+    void *q_abs = nullptr, *merged = nullptr;
     void* kv = nullptr;                                // expanded keys and values [batch][N][kv_row]
 };
 LatentState* latent(const b200p_session* s) { return static_cast<LatentState*>(s->decoder.get()); }
@@ -285,19 +285,29 @@ __global__ void __launch_bounds__(256) latent_norm_kernel(const LatentNormArgs a
     }
 }
 
-// Rotates the queries' rotated parts in place: one thread per pair.
+// Rotates the queries' rotated parts in place: a thread takes one group of eight pairs (16 columns) of a token and every
+// kRotHeads-th head.
+constexpr int kRotHeads = 4;
 template <typename T>
-__global__ void rotate_queries_kernel(T* __restrict__ q, const float* __restrict__ cos_t, const float* __restrict__ sin_t, LatentDims d,
-                                      int rows, int Tn, int pos0) {
+__global__ void __launch_bounds__(256) rotate_queries_kernel(T* __restrict__ q, const float* __restrict__ cos_t, const float* __restrict__ sin_t, LatentDims d,
+                                                             int rows, int Tn, int pos0) {
     const size_t i = size_t(blockIdx.x) * blockDim.x + threadIdx.x;
-    const int pairs = d.rot / 2;
-    if (i >= size_t(rows) * d.heads * pairs) return;
-    const int p = int(i % pairs), h = int(i / pairs % d.heads), r = int(i / pairs / d.heads);
-    T* v = q + size_t(r) * d.q_row() + size_t(h) * (d.dim + d.rot) + d.dim + 16 * (p / 8) + p % 8;
-    const size_t t = size_t(pos0 + r % Tn) * pairs + p;
-    const float c = cos_t[t], sn = sin_t[t], x0 = to_float(v[0]), x1 = to_float(v[8]);
-    v[0] = from_float<T>(x0 * c - x1 * sn);
-    v[8] = from_float<T>(x1 * c + x0 * sn);
+    const int groups = d.rot / 16;
+    if (i >= size_t(rows) * kRotHeads * groups) return;
+    const int gr = int(i % groups), h0 = int(i / groups % kRotHeads), r = int(i / groups / kRotHeads);
+    const size_t t = size_t(pos0 + r % Tn) * (d.rot / 2) + 8 * gr;
+    const float4 c[2] = {load4<float>(cos_t + t), load4<float>(cos_t + t + 4)}, sn[2] = {load4<float>(sin_t + t), load4<float>(sin_t + t + 4)};
+    T* v = q + size_t(r) * d.q_row() + d.dim + 16 * gr;
+    #pragma unroll 4
+    for (int h = h0; h < d.heads; h += kRotHeads) {
+        T* p = v + size_t(h) * (d.dim + d.rot);
+        #pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            const float4 x0 = load4<T>(p + 4 * k), x1 = load4<T>(p + 8 + 4 * k);
+            store4<T>(p + 4 * k, make_float4(x0.x * c[k].x - x1.x * sn[k].x, x0.y * c[k].y - x1.y * sn[k].y, x0.z * c[k].z - x1.z * sn[k].z, x0.w * c[k].w - x1.w * sn[k].w));
+            store4<T>(p + 8 + 4 * k, make_float4(x1.x * c[k].x + x0.x * sn[k].x, x1.y * c[k].y + x0.y * sn[k].y, x1.z * c[k].z + x0.z * sn[k].z, x1.w * c[k].w + x0.w * sn[k].w));
+        }
+    }
 }
 
 template <typename T>
@@ -336,7 +346,7 @@ int layers_gemm(b200p_session* s, int Tn, int pos0, cudaStream_t st) {
         if (int e = launched()) return e;
         // queries
         if (int e = session_gemm(s, L->cq, w.uq, L->q, M, qr, d.qrank, d.qrank, qr, f32, false, st)) return e;
-        rotate_queries_kernel<T><<<blocks(size_t(M) * d.heads * (d.rot / 2)), 256, 0, st>>>(static_cast<T*>(L->q), L->rot[li].first, L->rot[li].second, d, M, Tn, pos0);
+        rotate_queries_kernel<T><<<blocks(size_t(M) * kRotHeads * (d.rot / 16)), 256, 0, st>>>(static_cast<T*>(L->q), L->rot[li].first, L->rot[li].second, d, M, Tn, pos0);
         if (int e = launched()) return e;
         // keys and values of everything in the cache
         for (int b = 0; b < s->batch; ++b)
@@ -376,9 +386,18 @@ bool few_tokens(const b200p_session* s, int M) {
     return true;
 }
 
-// Nine launches a layer, each a programmatic dependent of the one before.  The norms on the sublayers' outputs and the
+// Ten launches a layer, each a programmatic dependent of the one before.  The norms on the sublayers' outputs and the
 // residual adds are prologues of whatever reads x next (PRO_POSTADD: every CTA forms the sum, CTA 0 keeps it in the other
-// of two buffers), so y and the norm's weights travel along as `pending`.
+// of two buffers), so y and the norm's weights travel along as `pending`.  With more rows than kFusedAddRows every CTA
+// would read too much fp32 for that: then the sum is a kernel of its own, which leaves x as 16-bit rows.
+constexpr int kFusedAddRows = 4;
+
+template <int EPI>
+int launch_reading_x(SkinnyArgs& a, bool fused, cudaStream_t st) {
+    using T = __nv_bfloat16;
+    return fused ? launch_skinny<T, PRO_POSTADD, EPI>(a, st) : launch_skinny<T, PRO_PLAIN, EPI>(a, st);
+}
+
 int layers_few(b200p_session* s, int Tn, int pos0, cudaStream_t st, const int* pos_dev) {
     using T = __nv_bfloat16;
     LatentState* L = latent(s);
@@ -392,7 +411,15 @@ int layers_few(b200p_session* s, int Tn, int pos0, cudaStream_t st, const int* p
         ++s->gemm_calls;
         return a;
     };
+    const bool fused = M <= kFusedAddRows;
     auto read_x = [&](SkinnyArgs& a) {                  // X = x + norm(pending)
+        if (!fused) {
+            postnorm_add_kernel<T><<<blocks(size_t(M) * 32), 256, 0, st>>>(x, pending, static_cast<const T*>(pending_w), static_cast<T*>(L->x16), M, H, n, s->eps);
+            launched();
+            a.X16 = L->x16; a.ldx = H;
+            pending = nullptr;
+            return;
+        }
         a.X32 = x; a.Y32 = pending; a.x_out = other; a.norm_w = pending_w; a.norm_n = n;
         if (pending) std::swap(x, other);
         pending = nullptr;
@@ -403,14 +430,14 @@ int layers_few(b200p_session* s, int Tn, int pos0, cudaStream_t st, const int* p
         const LatentDims d = ly.mix.dims();
         SkinnyArgs a = args(w.proj, L->proj, d.proj_row(), H, d.proj_row());
         read_x(a);
-        if (int e = launch_skinny<T, PRO_POSTADD, EPI_STORE32>(a, st)) return e;
+        if (int e = launch_reading_x<EPI_STORE32>(a, fused, st)) return e;
         a = args(w.uq, L->q, d.q_row(), d.qrank, d.heads * d.dim);
         a.X32 = L->proj; a.ldx32 = d.proj_row(); a.norm_w = w.q_norm; a.norm_n = ly.mix.q_rank;
         a.pair = SkinnyPairRot{L->rot[li].first, L->rot[li].second, pos_dev, L->q_abs, pos0, Tn, d.dim, d.rot, d.heads, d.cache_row(), d.rank, s->max_seq};
         if (int e = launch_skinny<T, PRO_RMSNORM, EPI_PAIRROT>(a, st)) return e;
         LatentStep p{d, s->batch, Tn, pos0, s->max_seq, pos_dev, float(ly.mix.scale), s->eps, ly.mix.kv_rank, w.sink, w.ukT,
                      static_cast<const T*>(w.kv) + size_t(d.heads) * d.dim * d.rank, w.kv_norm, L->rot[li].first, L->rot[li].second,
-                     L->proj, L->q, L->q_abs, L->cache[li], L->part_o, L->part_ml, L->attn, s->d_attn_status};
+                     L->proj, L->q, L->q_abs, L->cache[li], L->part_o, L->part_ml, L->merged, L->attn, s->d_attn_status};
         if (int e = latent_step_absorb(p, st)) return e;
         if (int e = latent_step_attend(p, st)) return e;
         if (int e = latent_step_values(p, st)) return e;
@@ -422,7 +449,7 @@ int layers_few(b200p_session* s, int Tn, int pos0, cudaStream_t st, const int* p
         const int F = pad16(ly.ff);
         a = args(w.gu, L->act, F, H, F);
         read_x(a);
-        if (int e = launch_skinny<T, PRO_POSTADD, EPI_GELU16>(a, st)) return e;
+        if (int e = launch_reading_x<EPI_GELU16>(a, fused, st)) return e;
         a = args(w.down, L->y, H, F, H);
         a.X16 = L->act; a.ldx = F;
         if (int e = launch_skinny<T, PRO_PLAIN, EPI_STORE32>(a, st)) return e;
@@ -615,6 +642,7 @@ int latent_build(b200p_session* s, const b200p_model* m) {
         if (cudaError_t e = s->alloc(&L->part_o, part_floats * 4)) return int(e);
         if (cudaError_t e = s->alloc(&L->part_ml, parts * 8)) return int(e);
         if (cudaError_t e = s->alloc(&L->q_abs, abs * 2)) return int(e);
+        if (cudaError_t e = s->alloc(&L->merged, abs * 2)) return int(e);
     }
     if (cudaError_t e = s->alloc(&s->d_attn_status, 16)) return int(e);
     return int(cudaMemset(s->d_attn_status, 0, 16));

@@ -38,6 +38,7 @@ from __future__ import annotations
 
 import argparse
 import json
+import math
 import os
 import statistics
 import sys
@@ -716,6 +717,152 @@ class RuntimeLlama:
 
 
 # --------------------------------------------------------------------------------------
+# workload: the decoder with latent attention (Maposun) in the runtime, beside the Llama-style one at equal width and depth
+# --------------------------------------------------------------------------------------
+class RuntimeLatent(RuntimeLlama):
+    name = "runtime_latent"
+    metric = "greedy generation throughput of the runtime, latent-attention decoder (generated tokens/s; prompt 512 + 128 new tokens)"
+    LAYERS = 22
+    # width, ff, latent mixer (heads, dim, rot_dim, vdim, kv_rank, q_rank), Llama attention (heads, kv heads, head dim)
+    SIZES = {"w1024": (1024, 2816, (8, 64, 32, 64, 256, 384), (16, 4, 64)),
+             "w2048": (2048, 5632, (16, 128, 64, 128, 512, 768), (32, 4, 64)),
+             "w4096": (4096, 14336, (32, 128, 64, 128, 512, 1536), (32, 8, 128))}
+    VOCAB = 32000
+    TABLE_LAYERS, TABLE_NEW = 8, 24
+    TABLE = [(1, 512), (1, 4096), (8, 4096)]   # sequences, prompt tokens
+    BASE = 10000.0
+
+    def __init__(self, n=None):
+        if n:
+            self.NEW = n
+        self.bytes_per_step = float(self.B * self.NEW)
+        self.cases = [("generate (prefill 512 + decode)", None, None, None, self.bytes_per_step)]
+        self.CFG = self.latent_config("w2048", self.LAYERS)
+        self.weight_bytes = 2 * sum(int(math.prod(s)) for k, s in self.latent_shapes(self.CFG).items() if k != "embed")
+
+    def latent_config(self, size, layers):
+        width, ff, (heads, dim, rot, vdim, kv, q), _ = self.SIZES[size]
+        mx = {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": vdim, "kv_rank": kv, "q_rank": q,
+              "rot": {"base": self.BASE, "dims": rot}, "scale": (dim + rot) ** -0.5}
+        return {"architecture": "Maposun", "width": width, "vocab": self.VOCAB, "norm": {"eps": 1e-6},
+                "layers": [{"type": "latent_attention_2" if i % 2 else "latent_attention", "mixer": mx, "mlp": {"kind": "dense", "ff": ff}}
+                           for i in range(layers)]}
+
+    @staticmethod
+    def latent_shapes(cfg):
+        out = {"embed": (cfg["vocab"], cfg["width"]), "final.norm": (cfg["width"],), "head": (cfg["vocab"], cfg["width"])}
+        for i, L in enumerate(cfg["layers"]):
+            m, D, p = L["mixer"], cfg["width"], f"l{i}."
+            H, ff = m["heads"], L["mlp"]["ff"]
+            out.update({p + "norm1": (D,), p + "norm2": (D,), p + "mix.dq": (m["q_rank"], D), p + "mix.dq.norm": (m["q_rank"],),
+                        p + "mix.uq": (H * (m["dim"] + m["rot_dim"]), m["q_rank"]), p + "mix.dkv": (m["kv_rank"] + m["rot_dim"], D),
+                        p + "mix.dkv.norm": (m["kv_rank"],), p + "mix.uk": (H * m["dim"], m["kv_rank"]), p + "mix.uv": (H * m["vdim"], m["kv_rank"]),
+                        p + "mix.g": (H * m["vdim"], D), p + "mix.o": (D, H * m["vdim"]),
+                        p + "mlp.gate": (ff, D), p + "mlp.up": (ff, D), p + "mlp.down": (D, ff)})
+            if L["type"] == "latent_attention_2":
+                out[p + "mix.sink"] = (H,)
+        return out
+
+    def config(self, world):
+        return {"workload": "latent-attention decoder (Maposun) in the runtime", "layers": self.LAYERS, "vocab": self.VOCAB,
+                "width": self.CFG["width"], "layer": self.CFG["layers"][0], "batch_per_gpu": self.B, "prompt_tokens": self.T, "new_tokens": self.NEW,
+                "sharding": f"sequences x{world} (2 per GPU), weights replicated, no collective",
+                "weights": "random-init bf16 ~ N(0, 0.02), norm weights 1", "inputs": "uniform random token ids, seeded",
+                "l2": "the weights (2 GB) are larger than L2"}
+
+    def latent_model(self, cfg):
+        torch = self.torch
+        g = torch.Generator(device=self.device); g.manual_seed(0xB205)
+        t = {}
+        for n, s in self.latent_shapes(cfg).items():
+            t[n] = (torch.ones(s, device=self.device) if "norm" in n else torch.randn(s, device=self.device, generator=g) * 0.02).bfloat16()
+        return self.pkg.Model.from_tensors(cfg, t)
+
+    def setup(self, torch, pkg, device, rank):
+        import numpy as np
+        self.torch, self.pkg, self.device = torch, pkg, device
+        self.sess = pkg.Session.from_model(self.latent_model(self.CFG), self.T + self.NEW, self.B)
+        self.ids = np.random.default_rng(0xB205 + rank).integers(0, self.VOCAB, (self.B, self.T)).astype(np.int32)
+        self.timings = []
+        torch.cuda.synchronize()
+
+    def extra(self):
+        import statistics as st
+        tt = [t[0] for t in self.timings[-5:]]; dd = [t[1] for t in self.timings[-5:]]
+        ms_tok = st.median(dd) / max(1, self.NEW - 1)
+        m = self.CFG["layers"][0]["mixer"]
+        kv_bytes = self.LAYERS * self.B * (self.T + self.NEW // 2) * (m["kv_rank"] + m["rot_dim"]) * 2
+        return {"ttft_ms": st.median(tt), "decode_ms_per_token": ms_tok, "decode_step_bytes": self.weight_bytes + kv_bytes,
+                "decode_hbm_GBs": (self.weight_bytes + kv_bytes) / (ms_tok * 1e-3) / 1e9, "gemm_calls_total": self.sess.gemm_calls}
+
+    def extra_fields(self):
+        """Prefill and decode throughput at a few layer sizes, and of the Llama-style decoder of the same width, depth and MLP."""
+        import gc
+        import numpy as np
+        torch, pkg = self.torch, self.pkg
+        del self.sess
+        gc.collect(); torch.cuda.empty_cache()
+        table = {}
+        for size, (width, ff, _, (heads, kvh, hd)) in self.SIZES.items():
+            for kind in ("maposun", "llama"):
+                if kind == "maposun":
+                    model = self.latent_model(self.latent_config(size, self.TABLE_LAYERS))
+                    make = lambda seq, b: pkg.Session.from_model(model, seq, b)
+                else:
+                    g = torch.Generator(device=self.device); g.manual_seed(1)
+                    w = lambda *shape: (torch.randn(shape, device=self.device, generator=g) * 0.02).bfloat16()
+                    ones = torch.ones(width, device=self.device, dtype=torch.bfloat16)
+                    qd, kvd = heads * hd, kvh * hd
+                    weights = {"embed_tokens": w(self.VOCAB, width), "lm_head": w(self.VOCAB, width), "final_norm": ones, "layers": [
+                        {"Wq": w(qd, width), "Wk": w(kvd, width), "Wv": w(kvd, width), "Wo": w(width, qd), "Wgate": w(ff, width), "Wup": w(ff, width),
+                         "Wdown": w(width, ff), "norm_attn": ones, "norm_mlp": ones} for _ in range(self.TABLE_LAYERS)]}
+                    c = dict(n_layers=self.TABLE_LAYERS, hidden=width, n_heads=heads, n_kv_heads=kvh, head_dim=hd, ffn_dim=ff, vocab_size=self.VOCAB,
+                             rope_theta=self.BASE)
+                    make = lambda seq, b: pkg.Session(c, weights, seq, b)
+                for b, T in self.TABLE:
+                    s = make(T + self.TABLE_NEW, b)
+                    ids = np.random.default_rng(1).integers(0, self.VOCAB, (b, T)).astype(np.int32)
+                    for _ in range(2):
+                        s.generate(ids, self.TABLE_NEW)
+                    tm = sorted(s.generate(ids, self.TABLE_NEW)[1] for _ in range(5))
+                    ttft = sorted(t[0] for t in tm)[2]; dec = sorted(t[1] for t in tm)[2] / (self.TABLE_NEW - 1)
+                    table.setdefault(f"{size}_batch{b}_prompt{T}", {})[kind] = {
+                        "prefill_tokens_per_s": round(b * T / ttft * 1e3), "prefill_us_per_layer": round(ttft * 1e3 / self.TABLE_LAYERS, 1),
+                        "decode_tokens_per_s": round(b / dec * 1e3), "decode_us_per_layer": round(dec * 1e3 / self.TABLE_LAYERS, 2)}
+                    s.close()
+                if kind == "maposun":
+                    model.close(); del model
+                else:
+                    del weights
+                gc.collect(); torch.cuda.empty_cache()
+        return {"sizes": table, "sizes_note": f"{self.TABLE_LAYERS} layers, {self.TABLE_NEW} new tokens; times include embedding, head and sampling; "
+                                              "llama: the Llama-style decoder of the same width and MLP"}
+
+    def cpu_run(self, orc, n, threads, reps=1):
+        """n = new tokens; prompt 32.  One random layer's matrices serve all layers."""
+        import numpy as np
+        from oracle import latent_ref as lr
+        if not hasattr(self, "_cpu_w"):
+            cfg = self.latent_config("w2048", 2)
+            rng = np.random.default_rng(5)
+            two = {k: (np.ones(s) if "norm" in k else rng.standard_normal(s, dtype=np.float32) * 0.02) for k, s in self.latent_shapes(cfg).items()}
+            full = json.loads(json.dumps(cfg))
+            full["layers"] = [dict(cfg["layers"][i % 2], **({"weights_of": i % 2} if i > 1 else {})) for i in range(self.LAYERS)]
+            self._cpu_w = (full, two)
+        ids = list(np.random.default_rng(1).integers(0, self.VOCAB, 32))
+        t0 = time.perf_counter()
+        for _ in range(reps):
+            seq = list(ids)
+            for _ in range(n):
+                seq.append(int(np.argmax(lr.forward(self._cpu_w[0], self._cpu_w[1], seq)[-1])))
+        dt = (time.perf_counter() - t0) / reps
+        return n / dt, dt
+
+    cpu_sample = 1
+    cpu_sample_text = "1 sequence, prompt 32 tokens + 1 new token (float64 numpy statement of the decoder)"
+
+
+# --------------------------------------------------------------------------------------
 # workload: the FA2 build-order steps at the reference's validation shape (BASELINE config 1)
 # --------------------------------------------------------------------------------------
 class FaSteps:
@@ -956,7 +1103,7 @@ class WaveApi:
 
 
 WORKLOADS = {"wave_api": WaveApi, "fa_steps": FaSteps, "segops": SegopsSweep, "decode": DecodeGQA, "prefill": PrefillCausal, "decode_long": DecodeLong,
-             "runtime": RuntimeLlama}
+             "runtime": RuntimeLlama, "runtime_latent": RuntimeLatent}
 ALL_ORDER = ["prefill", "decode", "segops", "decode_long", "runtime", "fa_steps", "wave_api"]   # `--workload all`: the first is the headline
 
 
@@ -1053,8 +1200,8 @@ def measure(wl, args, ctx):
         return float(t.item())
 
     wl.setup(torch, pkg, device, rank)
-    steps = args.steps if wl.name != "runtime" else max(2, min(args.steps, 5))     # a runtime step is a whole generation
-    warm = max(args.warmup, 3) if wl.name != "runtime" else 3
+    steps = args.steps if not wl.name.startswith("runtime") else max(2, min(args.steps, 5))     # a runtime step is a whole generation
+    warm = max(args.warmup, 3) if not wl.name.startswith("runtime") else 3
     for _ in range(warm):
         wl.step()
     barrier()
