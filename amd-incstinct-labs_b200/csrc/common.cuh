@@ -74,6 +74,19 @@ inline int launched(unsigned n = 1) {
 #ifdef __CUDACC__
 __device__ __forceinline__ void griddep_launch_dependents() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
 __device__ __forceinline__ void griddep_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
+// Launch as a programmatic dependent of the stream's previous kernel.
+template <typename... P, typename... A>
+int launch_dependent(void (*kern)(P...), dim3 grid, int threads, size_t smem, cudaStream_t st, A... args) {
+    cudaLaunchConfig_t cfg{};
+    cfg.gridDim = grid; cfg.blockDim = dim3(unsigned(threads)); cfg.dynamicSmemBytes = smem; cfg.stream = st;
+    cudaLaunchAttribute attr[1];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr; cfg.numAttrs = tuning(KNOB_RUNTIME_PDL, 1) != 0 ? 1 : 0;
+    const cudaError_t e = cudaLaunchKernelEx(&cfg, kern, args...);
+    g_launches.fetch_add(1, std::memory_order_relaxed);
+    return int(e);
+}
 #endif
 
 } // namespace b200p

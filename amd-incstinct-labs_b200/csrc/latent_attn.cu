@@ -128,20 +128,6 @@ constexpr int kAttendKeys = 64;
 constexpr float kNegBig = -1e30f;
 constexpr int kMaxSplits = 128;          // the merge reads up to four splits per lane
 
-// Launch as a programmatic dependent of the stream's previous kernel.
-template <typename... P, typename... A>
-int launch_dependent(void (*kern)(P...), dim3 grid, int threads, size_t smem, cudaStream_t st, A... args) {
-    cudaLaunchConfig_t cfg{};
-    cfg.gridDim = grid; cfg.blockDim = dim3(unsigned(threads)); cfg.dynamicSmemBytes = smem; cfg.stream = st;
-    cudaLaunchAttribute attr[1];
-    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[0].val.programmaticStreamSerializationAllowed = 1;
-    cfg.attrs = attr; cfg.numAttrs = tuning(KNOB_RUNTIME_PDL, 1) != 0 ? 1 : 0;
-    const cudaError_t e = cudaLaunchKernelEx(&cfg, kern, args...);
-    g_launches.fetch_add(1, std::memory_order_relaxed);
-    return int(e);
-}
-
 __device__ __forceinline__ int first_pos(const LatentStep& a) { return a.pos_dev ? min(*a.pos_dev, a.max_seq - a.Tn) : a.pos0; }
 
 // Sixteen rows of a weight matrix against X: the A fragments are 32 contiguous bytes of a row per lane (a dot product

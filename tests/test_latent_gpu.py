@@ -50,6 +50,8 @@ CONFIGS = {
     # the head sizes of the large models: the widest prefill and decode kernels
     "real_heads": config(256, 200, [("_2", REAL, 320), ("", REAL, 320)]),
     # key and value heads of different box counts
+    # an MLP too wide for the streaming kernels with eight rows and more
+    "wide_mlp": config(64, 70, [("", mixer(2, 16, 8, 16, 32, 32), 12304)]),
     "wide_keys": config(128, 96, [("", mixer(4, 96, 32, 48, 160, 64), 96), ("_2", mixer(4, 48, 64, 112, 272, 80), 96)]),
     # outside the tensor-core kernels' domain
     "too_wide": config(128, 96, [("", mixer(2, 144, 80, 160, 600, 64), 96), ("_2", mixer(2, 24, 16, 32, 528, 48), 96)]),
@@ -238,7 +240,7 @@ def test_cache_used_again(opened, dtype):
     assert np.array_equal(run(s, first, [200, 17, 1]), a)
 
 
-@pytest.mark.parametrize("name,dtype,batch", [("odd", "bf16", 3), ("odd", "f32", 2), ("many_heads", "bf16", 5), ("many_heads", "bf16", 20),
+@pytest.mark.parametrize("name,dtype,batch", [("odd", "bf16", 3), ("odd", "f32", 2), ("wide_mlp", "bf16", 8), ("many_heads", "bf16", 5), ("many_heads", "bf16", 20),
                                               ("real_heads", "bf16", 12)])
 def test_batch_against_each_alone(opened, name, dtype, batch):
     s = opened(name, dtype, max_seq=128, batch=batch)
