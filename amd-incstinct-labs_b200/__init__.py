@@ -1,5 +1,5 @@
-"""B200 (sm_100a) implementation of the reference's wave reduce/scan primitives and
-FA2 attention kernels: Python host layer over the C ABI of libb200p.so.
+"""B200 (sm_100a) implementation of the reference's wave reduce/scan primitives, FA2
+attention kernels and small LLM runtime: Python host layer over the C ABI of libb200p.so.
 
 The library is hand-written CUDA (csrc/) behind `extern "C"` entry points
 (include/b200p.h).  This module only loads it with ctypes and offers thin
@@ -530,11 +530,11 @@ class ModelWeights(C.Structure):
 def skinny_gemm(W, out, x16=None, x32=None, norm_w=None, epilogue: str = "store16", eps: float = 1e-6):
     """The decode step's projection kernel: out = X . W^T for at most 16 rows of X.
     X is x16 [M, K] (16-bit) or RMSNorm(x32 [M, K]) * norm_w; epilogue one of
-    store16 / store32 / acc32 (out += Y) / silu16 (W = [gate; up], out = SiLU(gate) * up)."""
-    epi = {"store16": 0, "acc32": 1, "store32": 2, "silu16": 3}[epilogue]
+    store16 / store32 / acc32 (out += Y) / silu16, gelu16 (W = [gate; up], out = act(gate) * up)."""
+    epi = {"store16": 0, "acc32": 1, "store32": 2, "silu16": 3, "gelu16": 6}[epilogue]
     _dev(W, "W"); _dev(out, "out")
     N, K = W.shape
-    if epi == 3:
+    if epi in (3, 6):
         N //= 2
     if x16 is not None:
         if not x16.is_cuda or x16.stride(1) != 1:
@@ -604,13 +604,13 @@ class Model:
 
 def gemm_16(A, W, out, epilogue: str = "store16"):
     """out[M, N] = A[M, K] . W[N, K]^T on the tensor cores; epilogue store16 / store32 / acc32 (out += product) /
-    silu16 (W = [gate; up] with 2N rows, out = SiLU(gate) * up).  A, W 16-bit CUDA tensors with contiguous rows."""
-    epi = {"store16": 0, "acc32": 1, "store32": 2, "silu16": 3}[epilogue]
+    silu16, gelu16 (W = [gate; up] with 2N rows, out = act(gate) * up).  A, W 16-bit CUDA tensors with contiguous rows."""
+    epi = {"store16": 0, "acc32": 1, "store32": 2, "silu16": 3, "gelu16": 6}[epilogue]
     for t, n in ((A, "A"), (W, "W"), (out, "out")):
         if not t.is_cuda or t.stride(-1) != 1:
             raise ValueError(f"{n} must be a CUDA tensor with contiguous rows: there is no CPU path")
     M, K = A.shape
-    N = W.shape[0] // (2 if epi == 3 else 1)
+    N = W.shape[0] // (2 if epi in (3, 6) else 1)
     _check(lib().b200p_gemm_16(_dtype_code(A), epi, A.data_ptr(), W.data_ptr(), out.data_ptr(), M, N, K,
                                A.stride(0), W.stride(0), out.stride(0), _stream(A)), "gemm_16")
     return out

@@ -128,8 +128,9 @@ void b200p_session_reset(b200p_session* s);
  *   prologue 1: X = RMSNorm(x32 [M, K] fp32) * norm_w, rounded to 16 bits (forward.hpp:34-56);
  *   epilogue 0: out 16-bit [M, ldo];  2: out fp32;  1: out fp32 += Y (residual);
  *   epilogue 3: W is [2N, K] (gate rows, then up rows), out 16-bit = SiLU(gate) * up
- *               (forward.hpp:154-160).
- * Combinations: prologue 1 with epilogues 0, 2, 3; prologue 0 with epilogue 1.
+ *               (forward.hpp:154-160);
+ *   epilogue 6: the same with the tanh form of GELU.
+ * Combinations: prologue 1 with epilogues 0, 2, 3; prologue 0 with epilogues 1, 2, 6.
  * K must be a multiple of 16; B200P_E_RANGE for shapes outside the kernel's domain. */
 int b200p_skinny_gemm(int dtype, int prologue, int epilogue, const void* W, const void* x16, const float* x32,
                       const void* norm_w, void* out, int M, int N, int K, int ldx, int ldo, float eps,
@@ -140,7 +141,8 @@ int b200p_skinny_gemm(int dtype, int prologue, int epilogue, const void* W, cons
  * Session::run_layers (rocblas_gemm.hpp:112-209; session.hpp:147-160,171-173,220,227-230) with the element-wise
  * kernel that follows each GEMM in the reference folded into the epilogue:
  *   epilogue 0: C 16-bit;  2: C fp32;  1: C fp32 += product (the residual add, forward.hpp add_f32_kernel);
- *   epilogue 3: W is [2N, K] (gate rows, then up rows), C 16-bit = SiLU(gate) * up (forward.hpp:154-160).
+ *   epilogue 3: W is [2N, K] (gate rows, then up rows), C 16-bit = SiLU(gate) * up (forward.hpp:154-160);
+ *   epilogue 6: the same with the tanh form of GELU.
  * A [M, lda] and W [N, ldw] 16-bit, row-major; lda, ldw, K multiples of 8; A, W, C and the rows of C 16-byte
  * aligned.  B200P_E_RANGE / B200P_E_ALIGN for anything else (nothing is launched). */
 int b200p_gemm_16(int dtype, int epilogue, const void* A, const void* W, void* C, int M, int N, int K,

@@ -40,6 +40,11 @@ public:
         if (!m_) throw std::runtime_error("ModelLoader: load() has not been called");
         return *b200p_model_weights_of(m_);
     }
+    // The loaded model, of any architecture the library knows (b200p_model_load).
+    const b200p_model* model() const {
+        if (!m_) throw std::runtime_error("ModelLoader: load() has not been called");
+        return m_;
+    }
 };
 
 // One sequence per session, like the reference's (batch = 1).
@@ -51,7 +56,7 @@ public:
     Session(const std::string& model_dir, int max_seq = 4096) : loader_(model_dir), max_seq_(max_seq) {
         loader_.load();
         int st = 0;
-        s_ = b200p_session_create(&loader_.weights(), max_seq, 1, &st);
+        s_ = b200p_session_open(loader_.model(), -1, max_seq, 1, &st);
         if (!s_) throw std::runtime_error(std::string("Session: ") + b200p_strerror(st));
     }
     Session(const Session&) = delete;
@@ -75,6 +80,16 @@ public:
         }
         return seq;
     }
+
+    // The next tokens on top of the cache (a prompt, a portion of one, or one token): fp32 logits of the wanted ones,
+    // [want.size()][vocab].  reset() starts a new sequence.
+    std::vector<float> extend(const std::vector<int>& tokens, const std::vector<int>& want) {
+        std::vector<float> logits(want.size() * size_t(config().vocab_size));
+        const int rc = b200p_session_extend(s_, tokens.data(), int(tokens.size()), want.data(), int(want.size()), logits.data(), nullptr);
+        if (rc) throw std::runtime_error(std::string("Session::extend: ") + b200p_strerror(rc));
+        return logits;
+    }
+    void reset() { b200p_session_reset(s_); }
 
     // Prefill only: fp32 logits of the last prompt token.
     std::vector<float> prefill_logits(const std::vector<int>& input_ids) {

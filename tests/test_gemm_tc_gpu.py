@@ -64,6 +64,21 @@ def test_silu_gate_up_epilogue(b200p, torch_cuda, M, F, K, kind):
     assert not out[:, F:].any()
 
 
+@pytest.mark.parametrize("M,F,K", [(300, 336, 208), (17, 16, 64), (128, 640, 512)])
+def test_gelu_epilogue(b200p, torch_cuda, M, F, K):
+    """out = gelu_tanh(gate) * up, gates from far negative to far positive."""
+    torch = torch_cuda
+    g = torch.Generator(device="cuda"); g.manual_seed(M)
+    A = (torch.randn(M, K, device="cuda", generator=g) * 1.5).bfloat16()
+    W = (torch.randn(2 * F, K, device="cuda", generator=g) / K ** 0.5 * 4).bfloat16()
+    gate, up = A.double() @ W[:F].double().T, A.double() @ W[F:].double().T
+    ref = torch.nn.functional.gelu(gate, approximate="tanh") * up
+    out = torch.zeros(M, F, dtype=torch.bfloat16, device="cuda")
+    b200p.gemm_16(A, W, out, "gelu16")
+    assert b200p.device_status() == 0
+    assert ((out.double() - ref).abs() < 2.0 ** -8 * ref.abs() + 2e-4).all()
+
+
 def test_domain_errors(b200p, torch_cuda):
     torch = torch_cuda
     A = torch.zeros(64, 36, dtype=torch.bfloat16, device="cuda")      # K not a multiple of 8

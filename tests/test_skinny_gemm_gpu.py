@@ -96,6 +96,22 @@ def test_silu_epilogue(b200p, torch_cuda, kind, M, F, K):
     assert np.abs(out.float().cpu().numpy() - ref).max() < (ulp + 3e-3) * max(1e-3, np.abs(ref).max())
 
 
+@pytest.mark.parametrize("M,F,K", [(2, 5632, 2048), (1, 40, 64), (11, 300, 512)])
+def test_gelu_epilogue_and_plain_store(b200p, torch_cuda, M, F, K):
+    torch = torch_cuda
+    rng = np.random.default_rng(F + M)
+    Wf, W = w16(torch, rng, (2 * F, K), "bf16", 3.0 / np.sqrt(K))
+    Xf, X = w16(torch, rng, (M, K), "bf16")
+    g, u = Xf @ Wf[:F].T, Xf @ Wf[F:].T
+    ref = 0.5 * g * (1.0 + np.tanh(np.sqrt(2 / np.pi) * (g + 0.044715 * g ** 3))) * u
+    out = torch.zeros((M, F), dtype=torch.bfloat16, device="cuda")
+    b200p.skinny_gemm(W, out, x16=X, epilogue="gelu16")
+    assert (np.abs(out.float().cpu().numpy() - ref) < 2.0 ** -8 * np.abs(ref) + 2e-4).all()
+    both = torch.zeros((M, 2 * F), dtype=torch.float32, device="cuda")
+    b200p.skinny_gemm(W, both, x16=X, epilogue="store32")
+    assert np.abs(both.cpu().numpy() - np.concatenate([g, u], 1)).max() < 1e-4 * max(1.0, np.abs(u).max())
+
+
 def test_shapes_outside_the_domain_are_refused(b200p, torch_cuda):
     torch = torch_cuda
     W = torch.zeros((64, 24), dtype=torch.bfloat16, device="cuda")          # K not a multiple of 16
