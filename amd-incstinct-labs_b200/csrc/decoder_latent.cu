@@ -2,7 +2,7 @@
 // decoder_latent.cu -- decoder with latent attention, gated attention output, norms on
 // the sublayers' outputs and a GELU-gated MLP: architecture "Maposun".
 //
-//   x <- x + norm1(mixer(x));  x <- x + norm2(mlp(x))        (the sublayers read x itself)
+//   y = x + N1(attention(x)),  z = y + N2(mlp(y))        (no norm in front of a sublayer)
 //
 // config.json lists the layers; each names its mixer type with the mixer's sizes and
 // its MLP (or none), and may use an earlier layer's tensors ("weights_of") with a cache

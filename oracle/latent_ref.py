@@ -1,6 +1,6 @@
 """Plain float64 statement of the decoder with latent attention and output norms (architecture "Maposun"), one
 function per mechanism.  Slow on purpose: whole sequences, one head at a time, no cache and no absorbed products.
-Used as the checker only; shares no code with the library.
+For tests and CPU timings only; shares no code with the library.
 
     x       residual stream, [tokens, width]
     config  the parsed config.json; weights: dict name -> array as stored in model.safetensors
@@ -9,7 +9,7 @@ import numpy as np
 
 
 def rms_norm(x, w, eps):
-    """x / sqrt(mean(x^2) + eps) * w over the last axis."""
+    """Over the last axis: x by the root of (mean square + eps), times w."""
     return x / np.sqrt(np.mean(x * x, axis=-1, keepdims=True) + eps) * w
 
 
@@ -69,12 +69,14 @@ def latent_attention(h, positions, mixer, kind, weights, prefix, eps):
     how = MIXERS[kind]
     H, dim, rot, vdim, rank = mixer["heads"], mixer["dim"], mixer["rot_dim"], mixer["vdim"], mixer["kv_rank"]
     T = h.shape[0]
-    ang = rotation_angles(positions, mixer["rot"]["dims"], mixer["rot"]["base"])
+    turning = mixer["rot"]["dims"]
+    ang = rotation_angles(positions, turning, mixer["rot"]["base"])
+    rotate = lambda v: np.concatenate([how["rotate"](v[..., :turning], ang), v[..., turning:]], axis=-1)
     q = (rms_norm(h @ W("dq").T, W("dq.norm"), eps) @ W("uq").T).reshape(T, H, dim + rot)
-    q_plain, q_rot = q[..., :dim], how["rotate"](q[..., dim:], ang)
+    q_plain, q_rot = q[..., :dim], rotate(q[..., dim:])
     down = h @ W("dkv").T
     latent = rms_norm(down[:, :rank], W("dkv.norm"), eps)
-    k_rot = how["rotate"](down[:, rank:], ang)                       # one for all heads
+    k_rot = rotate(down[:, rank:])                       # one for all heads
     k_plain = (latent @ W("uk").T).reshape(T, H, dim)
     v = (latent @ W("uv").T).reshape(T, H, vdim)
     visible = np.asarray(positions)[None, :] <= np.asarray(positions)[:, None]

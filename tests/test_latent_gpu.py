@@ -20,9 +20,9 @@ ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 BAR = {"f32": 1e-4, "bf16": 0.06}
 
 
-def mixer(heads, dim, rot, vdim, kv, q, base=10000.0, scale=None):
+def mixer(heads, dim, rot, vdim, kv, q, base=10000.0, scale=None, turning=None):
     return {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": vdim, "kv_rank": kv, "q_rank": q,
-            "rot": {"base": base, "dims": rot}, "scale": scale or 1.5 / np.sqrt(dim + rot)}
+            "rot": {"base": base, "dims": rot if turning is None else turning}, "scale": scale or 1.5 / np.sqrt(dim + rot)}
 
 
 def config(width, vocab, layers, eps=1e-5):
@@ -40,7 +40,7 @@ ODD = mixer(5, 24, 12, 40, 72, 56, 500.0)
 ODD2 = mixer(3, 40, 6, 22, 100, 36)
 ONE = mixer(1, 16, 2, 16, 16, 16, 3.0)
 MANY = mixer(20, 16, 16, 16, 48, 32)
-REAL = mixer(16, 128, 64, 128, 512, 96)
+REAL = mixer(16, 128, 64, 128, 512, 112)
 CONFIGS = {
     # nothing a multiple of 16, layers without MLP, shared layers, both mixers with different sizes
     "odd": config(200, 333, [("", ODD, 168), ("_2", ODD2, None), ("", ODD, 168, 0), ("_2", ODD2, None, 1), ("_2", ODD, 100)], 1e-3),
@@ -48,11 +48,13 @@ CONFIGS = {
     # more query rows than one 16-row tile for a single token
     "many_heads": config(96, 130, [("_2", MANY, 64), ("", MANY, None), ("", MANY, 64)]),
     # the head sizes of the large models: the widest prefill and decode kernels
-    "real_heads": config(256, 200, [("_2", REAL, 320), ("", REAL, 320)]),
+    "real_heads": config(288, 200, [("_2", REAL, 352), ("", REAL, 352)]),
     # key and value heads of different box counts
     # an MLP too wide for the streaming kernels with eight rows and more
     "wide_mlp": config(64, 70, [("", mixer(2, 16, 8, 16, 32, 32), 12304)]),
     "wide_keys": config(128, 96, [("", mixer(4, 96, 32, 48, 160, 64), 96), ("_2", mixer(4, 48, 64, 112, 272, 80), 96)]),
+    # rotated parts of which only the first dimensions turn, an odd number among them
+    "partly_rotated": config(80, 60, [("", mixer(3, 32, 20, 32, 48, 40, 50.0, turning=8), 64), ("_2", mixer(2, 16, 13, 16, 32, 32, 50.0, turning=10), 64)]),
     # outside the tensor-core kernels' domain
     "too_wide": config(128, 96, [("", mixer(2, 144, 80, 160, 600, 64), 96), ("_2", mixer(2, 24, 16, 32, 528, 48), 96)]),
 }
@@ -183,7 +185,7 @@ def test_key_tiles_edges_in_decoding(opened):
 def test_far_keys(opened, dtype, sharp):
     """One layer, sharp scores: most rows have one key that takes nearly everything, hundreds of tokens back for many.
     The oracle's own weights say so, and the logits follow."""
-    mx = mixer(2, 32, 16, 32, 64, 48, 1e4, sharp * 1.5 / np.sqrt(48))
+    mx = mixer(2, 40, 24, 24, 64, 48, 1e4, sharp * 1.5 / np.sqrt(64))
     cfg = config(96, 120, [("", mx, None)])
     name = "far%g" % sharp
     ids = tokens(cfg, 600, 4)
@@ -199,7 +201,7 @@ def test_far_keys(opened, dtype, sharp):
 @pytest.mark.parametrize("dtype", ["f32", "bf16"])
 def test_sinks(opened, dtype):
     """Sinks from nothing to everything: a layer whose sinks are left out, scaled or counted per key differs grossly."""
-    cfg = config(96, 120, [("_2", mixer(6, 32, 16, 32, 64, 48), None)])
+    cfg = config(96, 120, [("_2", mixer(6, 40, 24, 24, 64, 48), None)])
     name = "sinks"
     w = weights(name, cfg)
     ids = tokens(cfg, 140, 5)
