@@ -22,7 +22,7 @@ __device__ __forceinline__ float fast_exp2(float x) {
     return y;
 }
 
-// max of three (one FMNMX3 on sm_100a)
+// max of three (the three-input form of PTX max.f32)
 __device__ __forceinline__ float max3(float a, float b, float c) {
     float r;
     asm("max.f32 %0, %1, %2, %3;" : "=f"(r) : "f"(a), "f"(b), "f"(c));
