@@ -30,7 +30,8 @@ NVCC_FLAGS = [
 
 # the sources every decoder of the runtime needs, and each decoder's own
 RUNTIME = ("core", "tensor_map", "gemm_tc", "model_loader", "runtime")
-DECODERS = {"Llama": ("decoder_gqa", "decode", "prefill"), "Maposun": ("decoder_latent", "latent_attn", "latent_prefill")}
+DECODERS = {"Llama": ("decoder_gqa", "decode", "prefill"), "Maposun": ("decoder_latent", "latent_attn", "latent_prefill"),
+            "Vofusun": ("decoder_hybrid", "grouped_attn", "grouped_prefill", "delta_rule")}
 
 
 def _newest_header() -> float:

@@ -41,4 +41,14 @@ __device__ __forceinline__ float2 exp2_pair(float a, float b, float scale, float
     return make_float2(fast_exp2(lo), fast_exp2(hi));
 }
 
+// Which keys at or before its own position p a query sees: all of them, the last `size` (itself among them), or those of
+// its chunk of `size` positions counted from the sequence's start.
+enum AttnMaskKind { MASK_CAUSAL = 0, MASK_WINDOW = 1, MASK_CHUNK = 2 };
+struct AttnMask {
+    int kind, size;
+    __host__ __device__ int first(int p) const {
+        return kind == MASK_WINDOW ? (p - size + 1 > 0 ? p - size + 1 : 0) : kind == MASK_CHUNK ? p / size * size : 0;
+    }
+};
+
 } // namespace b200p

@@ -36,6 +36,8 @@ enum Knob {
     KNOB_RUNTIME_MEGA,          // 1: the greedy loop's decode steps run as one persistent cooperative kernel, 0: kernel per phase (default)
     KNOB_RUNTIME_MEGA_AHEAD,    // persistent decode kernel: stages of L2 prefetch in front of the shared-memory ring's loads
     KNOB_LATENT_PLAIN,          // 1: latent attention of 16-bit sessions on the plain kernel as well
+    KNOB_GROUPED_PLAIN,         // 1: grouped attention of 16-bit sessions on the plain kernel as well
+    KNOB_DELTA_PLAIN,           // 1: the gated delta rule token by token on the plain kernel
     KNOB_COUNT
 };
 
@@ -74,18 +76,31 @@ inline int launched(unsigned n = 1) {
 #ifdef __CUDACC__
 __device__ __forceinline__ void griddep_launch_dependents() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
 __device__ __forceinline__ void griddep_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
-// Launch as a programmatic dependent of the stream's previous kernel.
+// Launch as a programmatic dependent of the stream's previous kernel, in clusters of `cluster` CTAs along x (0: none).
 template <typename... P, typename... A>
-int launch_dependent(void (*kern)(P...), dim3 grid, int threads, size_t smem, cudaStream_t st, A... args) {
+int launch_dependent_clusters(void (*kern)(P...), int cluster, dim3 grid, int threads, size_t smem, cudaStream_t st, A... args) {
     cudaLaunchConfig_t cfg{};
     cfg.gridDim = grid; cfg.blockDim = dim3(unsigned(threads)); cfg.dynamicSmemBytes = smem; cfg.stream = st;
-    cudaLaunchAttribute attr[1];
-    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[0].val.programmaticStreamSerializationAllowed = 1;
-    cfg.attrs = attr; cfg.numAttrs = tuning(KNOB_RUNTIME_PDL, 1) != 0 ? 1 : 0;
+    cudaLaunchAttribute attr[2];
+    int n = 0;
+    if (cluster > 0) {
+        attr[n].id = cudaLaunchAttributeClusterDimension;
+        attr[n].val.clusterDim.x = unsigned(cluster); attr[n].val.clusterDim.y = attr[n].val.clusterDim.z = 1;
+        ++n;
+    }
+    if (tuning(KNOB_RUNTIME_PDL, 1) != 0) {
+        attr[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+        attr[n].val.programmaticStreamSerializationAllowed = 1;
+        ++n;
+    }
+    cfg.attrs = attr; cfg.numAttrs = unsigned(n);
     const cudaError_t e = cudaLaunchKernelEx(&cfg, kern, args...);
     g_launches.fetch_add(1, std::memory_order_relaxed);
     return int(e);
+}
+template <typename... P, typename... A>
+int launch_dependent(void (*kern)(P...), dim3 grid, int threads, size_t smem, cudaStream_t st, A... args) {
+    return launch_dependent_clusters(kern, 0, grid, threads, smem, st, args...);
 }
 #endif
 

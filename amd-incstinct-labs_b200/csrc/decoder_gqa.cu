@@ -84,17 +84,6 @@ __global__ void rope_scatter_kernel(T* __restrict__ qkv, const T* __restrict__ b
     }
 }
 
-// forward.hpp:154-160: silu(gate) * up in fp32, written as the down projection's 16-bit operand.
-// gu is [M, 2F]: gate in the first F columns, up in the last F.
-template <typename T>
-__global__ void silu_mul_cast_kernel(const float* __restrict__ gu, T* __restrict__ act, size_t M, int F) {
-    const size_t i = size_t(blockIdx.x) * blockDim.x + threadIdx.x;
-    if (i >= M * F) return;
-    const size_t m = i / F; const int f = int(i % F);
-    const float g = gu[m * 2 * F + f], u = gu[m * 2 * F + F + f];
-    act[i] = from_float<T>((g / (1.f + expf(-g))) * u);
-}
-
 template <typename T>
 __global__ void concat_rows_kernel(T* __restrict__ dst, const T* __restrict__ a, size_t na, const T* __restrict__ b, size_t nb,
                                    const T* __restrict__ c, size_t nc) {

@@ -23,9 +23,9 @@
 #include "session.cuh"
 #include "latent.cuh"
 #include "model.hpp"
+#include "weights.cuh"
 #include <algorithm>
 #include <cmath>
-#include <functional>
 #include <map>
 #include <string>
 #include <tuple>
@@ -60,19 +60,6 @@ struct LatentSpec {
     double eps = 0.0;
     std::vector<LatentLayer> layers;
 };
-
-bool read_int(const Json* obj, const char* key, int* out, int least = 1) {
-    const Json* v = obj ? obj->get(key) : nullptr;
-    if (!v || !v->is_int() || v->num < least || v->num > 1e9) return false;
-    *out = int(v->num);
-    return true;
-}
-bool read_num(const Json* obj, const char* key, double* out) {
-    const Json* v = obj ? obj->get(key) : nullptr;
-    if (!v || v->kind != Json::Number) return false;
-    *out = v->num;
-    return true;
-}
 
 int latent_configure(b200p_model* m, std::vector<TensorWant>* want) {
     auto spec = std::make_shared<LatentSpec>();
@@ -140,45 +127,6 @@ int latent_configure(b200p_model* m, std::vector<TensorWant>* want) {
 }
 
 // ---- packed weights -------------------------------------------------------------------------------
-// Element (r, c) of a stored matrix goes to dst[row_at[r] + col_at[c]].
-template <typename T>
-__global__ void pack_kernel(T* __restrict__ dst, const void* __restrict__ src, int src_dtype, int rows, int cols,
-                            const long long* __restrict__ row_at, const long long* __restrict__ col_at) {
-    const size_t n = size_t(rows) * cols;
-    for (size_t i = size_t(blockIdx.x) * blockDim.x + threadIdx.x; i < n; i += size_t(gridDim.x) * blockDim.x) {
-        const int r = int(i / cols), c = int(i % cols);
-        const float v = src_dtype == B200P_BF16 ? to_float(static_cast<const __nv_bfloat16*>(src)[i])
-                      : src_dtype == B200P_F16  ? to_float(static_cast<const __half*>(src)[i]) : static_cast<const float*>(src)[i];
-        dst[row_at[r] + col_at[c]] = from_float<T>(v);
-    }
-}
-
-using Where = std::function<long long(int)>;
-
-template <typename T> int type_code();
-template <> int type_code<float>() { return B200P_F32; }
-template <> int type_code<__nv_bfloat16>() { return B200P_BF16; }
-
-template <typename T>
-int pack(T* dst, const TensorRef& t, const Where& row_at, const Where& col_at) {
-    const int rows = t.shape.size() > 1 ? int(t.shape[0]) : 1, cols = int(t.shape.back());
-    if (t.dtype != B200P_BF16 && t.dtype != B200P_F16 && t.dtype != B200P_F32) return B200P_E_DTYPE;
-    std::vector<long long> at(size_t(rows) + cols);
-    for (int r = 0; r < rows; ++r) at[r] = row_at(r);
-    for (int c = 0; c < cols; ++c) at[size_t(rows) + c] = col_at(c);
-    long long* dev = nullptr;
-    if (cudaError_t e = cudaMalloc(&dev, at.size() * sizeof(long long))) return int(e);
-    cudaError_t e = cudaMemcpy(dev, at.data(), at.size() * sizeof(long long), cudaMemcpyHostToDevice);
-    if (e == cudaSuccess) {
-        const size_t n = size_t(rows) * cols;
-        pack_kernel<T><<<unsigned(std::min<size_t>((n + 255) / 256, 8192)), 256>>>(dst, t.dev, t.dtype, rows, cols, dev, dev + rows);
-        const int rc = launched();
-        e = rc ? cudaError_t(rc) : cudaDeviceSynchronize();
-    }
-    cudaFree(dev);
-    return int(e);
-}
-
 // The tensors of one layer, packed and padded (T elements except the sink).
 struct LatentWeights {
     void *proj = nullptr, *uq = nullptr, *kv = nullptr, *ukT = nullptr, *o = nullptr, *gu = nullptr, *down = nullptr;
@@ -525,28 +473,13 @@ int build_weights(b200p_session* s, const b200p_model* m) {
     LatentState* L = latent(s);
     const LatentSpec& spec = L->spec;
     const int H = L->H;
-    int rc = B200P_OK;
-    auto zeros = [&](size_t n, size_t esz) -> void* {
-        void* p = nullptr;
-        if (rc) return nullptr;
-        if (cudaError_t e = s->alloc(&p, n * esz)) { rc = int(e); return nullptr; }
-        if (cudaError_t e = cudaMemset(p, 0, n * esz)) { rc = int(e); return nullptr; }
-        return p;
-    };
-    auto put = [&](void* dst, const std::string& name, const Where& row_at, const Where& col_at) {
-        if (!rc) rc = pack<T>(static_cast<T*>(dst), m->tensors.at(name), row_at, col_at);
-    };
-    const Where same = [](int i) -> long long { return i; };
-    auto stride = [](long long ld, long long first = 0) -> Where { return [=](int i) { return (first + i) * ld; }; };
-    // a whole matrix or vector whose rows only need padding to `ld` columns (and `rows_p` rows); as it is when they need none
-    auto padded = [&](const std::string& name, int rows_p, int ld) -> void* {
-        const TensorRef& t = m->tensors.at(name);
-        const int rows = t.shape.size() > 1 ? int(t.shape[0]) : 1;
-        if (t.dtype == type_code<T>() && rows == rows_p && t.shape.back() == ld && aligned(t.dev, 32)) return const_cast<void*>(t.dev);
-        void* p = zeros(size_t(rows_p) * ld, sizeof(T));
-        put(p, name, stride(ld), same);
-        return p;
-    };
+    WeightPacker<T> pk{s, m};
+    int& rc = pk.rc;
+    auto zeros = [&](size_t n, size_t esz) { return pk.zeros(n, esz); };
+    auto put = [&](void* dst, const std::string& name, const Where& row_at, const Where& col_at) { pk.put(dst, name, row_at, col_at); };
+    auto padded = [&](const std::string& name, int rows_p, int ld) { return pk.padded(name, rows_p, ld); };
+    const Where same = at_index();
+    auto stride = [](long long ld, long long first = 0) { return at_stride(ld, first); };
     s->embed = padded("embed", spec.vocab, H);
     s->lm_head = padded("head", spec.vocab, H);
     s->final_norm = padded("final.norm", 1, H);
@@ -607,21 +540,11 @@ int build_weights(b200p_session* s, const b200p_model* m) {
     return rc;
 }
 
-// cos and sin of p * base^(-2i / dims), [max_seq][rot / 2]; pairs past dims / 2 do not turn.  Angles in double.
+// Angles p * base^(-2i / dims), [max_seq][rot / 2]; pairs past dims / 2 do not turn.
 int build_rotation(b200p_session* s, const LatentMixer& x, std::pair<float*, float*>* out) {
-    const int pairs = x.dims().rot / 2;
-    std::vector<float> c(size_t(s->max_seq) * pairs, 1.f), sn(c.size(), 0.f);
-    for (int i = 0; i < x.rot_dims / 2; ++i) {
-        const double f = std::pow(x.rot_base, -2.0 * i / x.rot_dims);
-        for (int p = 0; p < s->max_seq; ++p) {
-            c[size_t(p) * pairs + i] = float(std::cos(p * f));
-            sn[size_t(p) * pairs + i] = float(std::sin(p * f));
-        }
-    }
-    cudaError_t e;
-    if ((e = s->alloc(&out->first, c.size() * 4)) || (e = s->alloc(&out->second, c.size() * 4))) return int(e);
-    if ((e = cudaMemcpy(out->first, c.data(), c.size() * 4, cudaMemcpyHostToDevice))) return int(e);
-    return int(cudaMemcpy(out->second, sn.data(), c.size() * 4, cudaMemcpyHostToDevice));
+    std::vector<double> f;
+    for (int i = 0; i < x.rot_dims / 2; ++i) f.push_back(std::pow(x.rot_base, -2.0 * i / x.rot_dims));
+    return rotation_table(s, f, x.dims().rot / 2, out);
 }
 
 template <typename T> const DecoderOps* latent_ops() {

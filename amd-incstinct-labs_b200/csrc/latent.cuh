@@ -21,8 +21,6 @@
 
 namespace b200p {
 
-inline int pad16(int n) { return (n + 15) / 16 * 16; }
-
 struct LatentDims {
     int heads, dim, rot, vdim, rank, qrank;       // padded; rot holds whole groups of 8 pairs (see SkinnyPairRot)
     __host__ __device__ int cache_row() const { return rank + rot; }

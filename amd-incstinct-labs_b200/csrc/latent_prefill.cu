@@ -4,30 +4,11 @@
 // ---------------------------------------------------------------------------
 #include "latent.cuh"
 #include "prefill_tc.cuh"
+#include "gate_rows.cuh"
 #include "b200p.h"
 
 namespace b200p {
 namespace {
-
-// out *= sigmoid(gate), eight columns per thread.
-template <typename T>
-__global__ void __launch_bounds__(256) gate_kernel(T* __restrict__ out, const float* __restrict__ gate, size_t rows, int cols, int gate_ld) {
-    const size_t i = size_t(blockIdx.x) * blockDim.x + threadIdx.x;
-    const int per_row = cols / 8;
-    if (i >= rows * per_row) return;
-    const size_t r = i / per_row;
-    const int c = int(i % per_row) * 8;
-    uint4 v = *reinterpret_cast<const uint4*>(out + r * cols + c);
-    const float4* g = reinterpret_cast<const float4*>(gate + r * gate_ld + c);
-    const float4 g0 = g[0], g1 = g[1];
-    const float gf[8] = {g0.x, g0.y, g0.z, g0.w, g1.x, g1.y, g1.z, g1.w};
-    const T* e = reinterpret_cast<const T*>(&v);
-    float o[8];
-    #pragma unroll
-    for (int k = 0; k < 8; ++k) o[k] = to_float(e[k]) / (1.f + __expf(-gf[k]));
-    v = make_uint4(pack2<T>(o[0], o[1]), pack2<T>(o[2], o[3]), pack2<T>(o[4], o[5]), pack2<T>(o[6], o[7]));
-    *reinterpret_cast<uint4*>(out + r * cols + c) = v;
-}
 
 template <typename T, int PLAIN, int VS>
 int launch(const LatentAttn& a, cudaStream_t st) {
@@ -67,9 +48,7 @@ int launch(const LatentAttn& a, cudaStream_t st) {
     const int sms = sm_count();
     kern<<<unsigned(items < sms ? items : sms), prefill_threads(1), Sh::SMEM_BYTES, st>>>(p, mq, mk, mv, mo, mqr, mkr);
     if (int le = launched()) return le;
-    const size_t n = size_t(a.batch) * a.Tn * (vrow / 8);
-    gate_kernel<T><<<unsigned((n + 255) / 256), 256, 0, st>>>(static_cast<T*>(a.out), a.proj + d.gate_col(), size_t(a.batch) * a.Tn, int(vrow), d.proj_row());
-    return launched();
+    return gate_rows(static_cast<T*>(a.out), a.proj + d.gate_col(), size_t(a.batch) * a.Tn, int(vrow), d.proj_row(), st);
 }
 
 } // namespace

@@ -26,15 +26,18 @@ namespace b200p {
 namespace {
 
 // ---- kernels ------------------------------------------------------------------------------
-// forward.hpp:174-183: out[t, :] = float(embed[ids[t], :])
+// forward.hpp:174-183: out[t, :] = float(embed[ids[t], :]), times a scale, and once more to `copy` if it is given
 template <typename T>
-__global__ void embed_gather_kernel(const T* __restrict__ embed, const int* __restrict__ ids, float* __restrict__ out, int M, int H) {
+__global__ void embed_gather_kernel(const T* __restrict__ embed, const int* __restrict__ ids, float* __restrict__ out, float* __restrict__ copy, float scale, int M, int H) {
     griddep_launch_dependents();
     const int t = blockIdx.x;
     if (t >= M) return;
     const T* src = embed + size_t(ids[t]) * H;
-    float* dst = out + size_t(t) * H;
-    for (int i = threadIdx.x; i < H; i += blockDim.x) dst[i] = to_float(src[i]);
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+        const float v = to_float(src[i]) * scale;
+        out[size_t(t) * H + i] = v;
+        if (copy) copy[size_t(t) * H + i] = v;
+    }
 }
 
 // forward.hpp:244-262 argmax over a [V] row of 16-bit logits; ties go to the lowest index.
@@ -225,7 +228,7 @@ int last_logits_step(b200p_session* s, cudaStream_t st) {
 int embed(b200p_session* s, const int* ids, int M, cudaStream_t st) {
     return with_type(s->dtype, [&](auto tag) -> int {
         using T = decltype(tag);
-        embed_gather_kernel<T><<<M, 256, 0, st>>>(static_cast<const T*>(s->embed), ids, s->hidden, M, s->H);
+        embed_gather_kernel<T><<<M, 256, 0, st>>>(static_cast<const T*>(s->embed), ids, s->hidden, s->embedded, s->embed_scale, M, s->H);
         return launched();
     });
 }
