@@ -731,16 +731,17 @@ class RuntimeLatent(RuntimeLlama):
     TABLE_LAYERS, TABLE_NEW = 8, 24
     TABLE = [(1, 512), (1, 4096), (8, 4096)]   # sequences, prompt tokens
     BASE = 10000.0
+    KINDS = ("maposun",)                       # rows of the table beside "llama"
 
     def __init__(self, n=None):
         if n:
             self.NEW = n
         self.bytes_per_step = float(self.B * self.NEW)
         self.cases = [("generate (prefill 512 + decode)", None, None, None, self.bytes_per_step)]
-        self.CFG = self.latent_config("w2048", self.LAYERS)
-        self.weight_bytes = 2 * sum(int(math.prod(s)) for k, s in self.latent_shapes(self.CFG).items() if k != "embed")
+        self.CFG = self.own_config("w2048", self.LAYERS)
+        self.weight_bytes = 2 * sum(int(math.prod(s)) for k, s in self.own_shapes(self.CFG).items() if k != "embed")
 
-    def latent_config(self, size, layers):
+    def own_config(self, size, layers, kind=None):
         width, ff, (heads, dim, rot, vdim, kv, q), _ = self.SIZES[size]
         mx = {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": vdim, "kv_rank": kv, "q_rank": q,
               "rot": {"base": self.BASE, "dims": rot}, "scale": (dim + rot) ** -0.5}
@@ -749,7 +750,7 @@ class RuntimeLatent(RuntimeLlama):
                            for i in range(layers)]}
 
     @staticmethod
-    def latent_shapes(cfg):
+    def own_shapes(cfg):
         out = {"embed": (cfg["vocab"], cfg["width"]), "final.norm": (cfg["width"],), "head": (cfg["vocab"], cfg["width"])}
         for i, L in enumerate(cfg["layers"]):
             m, D, p = L["mixer"], cfg["width"], f"l{i}."
@@ -770,18 +771,18 @@ class RuntimeLatent(RuntimeLlama):
                 "weights": "random-init bf16 ~ N(0, 0.02), norm weights 1", "inputs": "uniform random token ids, seeded",
                 "l2": "the weights (2 GB) are larger than L2"}
 
-    def latent_model(self, cfg):
+    def own_model(self, cfg):
         torch = self.torch
         g = torch.Generator(device=self.device); g.manual_seed(0xB205)
         t = {}
-        for n, s in self.latent_shapes(cfg).items():
+        for n, s in self.own_shapes(cfg).items():
             t[n] = (torch.ones(s, device=self.device) if "norm" in n else torch.randn(s, device=self.device, generator=g) * 0.02).bfloat16()
         return self.pkg.Model.from_tensors(cfg, t)
 
     def setup(self, torch, pkg, device, rank):
         import numpy as np
         self.torch, self.pkg, self.device = torch, pkg, device
-        self.sess = pkg.Session.from_model(self.latent_model(self.CFG), self.T + self.NEW, self.B)
+        self.sess = pkg.Session.from_model(self.own_model(self.CFG), self.T + self.NEW, self.B)
         self.ids = np.random.default_rng(0xB205 + rank).integers(0, self.VOCAB, (self.B, self.T)).astype(np.int32)
         self.timings = []
         torch.cuda.synchronize()
@@ -804,9 +805,9 @@ class RuntimeLatent(RuntimeLlama):
         gc.collect(); torch.cuda.empty_cache()
         table = {}
         for size, (width, ff, _, (heads, kvh, hd)) in self.SIZES.items():
-            for kind in ("maposun", "llama"):
-                if kind == "maposun":
-                    model = self.latent_model(self.latent_config(size, self.TABLE_LAYERS))
+            for kind in (*self.KINDS, "llama"):
+                if kind != "llama":
+                    model = self.own_model(self.own_config(size, self.TABLE_LAYERS, kind))
                     make = lambda seq, b: pkg.Session.from_model(model, seq, b)
                 else:
                     g = torch.Generator(device=self.device); g.manual_seed(1)
@@ -830,7 +831,7 @@ class RuntimeLatent(RuntimeLlama):
                         "prefill_tokens_per_s": round(b * T / ttft * 1e3), "prefill_us_per_layer": round(ttft * 1e3 / self.TABLE_LAYERS, 1),
                         "decode_tokens_per_s": round(b / dec * 1e3), "decode_us_per_layer": round(dec * 1e3 / self.TABLE_LAYERS, 2)}
                     s.close()
-                if kind == "maposun":
+                if kind != "llama":
                     model.close(); del model
                 else:
                     del weights
@@ -843,9 +844,9 @@ class RuntimeLatent(RuntimeLlama):
         import numpy as np
         from oracle import latent_ref as lr
         if not hasattr(self, "_cpu_w"):
-            cfg = self.latent_config("w2048", 2)
+            cfg = self.own_config("w2048", 2)
             rng = np.random.default_rng(5)
-            two = {k: (np.ones(s) if "norm" in k else rng.standard_normal(s, dtype=np.float32) * 0.02) for k, s in self.latent_shapes(cfg).items()}
+            two = {k: (np.ones(s) if "norm" in k else rng.standard_normal(s, dtype=np.float32) * 0.02) for k, s in self.own_shapes(cfg).items()}
             full = json.loads(json.dumps(cfg))
             full["layers"] = [dict(cfg["layers"][i % 2], **({"weights_of": i % 2} if i > 1 else {})) for i in range(self.LAYERS)]
             self._cpu_w = (full, two)
@@ -860,6 +861,80 @@ class RuntimeLatent(RuntimeLlama):
 
     cpu_sample = 1
     cpu_sample_text = "1 sequence, prompt 32 tokens + 1 new token (float64 numpy statement of the decoder)"
+
+
+# --------------------------------------------------------------------------------------
+# workload: the decoder with gated-delta-rule layers and masked attention (Vofusun), beside the Llama-style one at equal width
+# --------------------------------------------------------------------------------------
+class RuntimeHybrid(RuntimeLatent):
+    name = "runtime_hybrid"
+    metric = "greedy generation throughput of the runtime, decoder with delta-rule and masked-attention layers (generated tokens/s; prompt 512 + 128 new tokens)"
+    LAYERS = 24
+    # width, ff, ((delta heads, kv heads, dim), (attention heads, kv heads, dim)), Llama attention (heads, kv heads, head dim)
+    SIZES = {"w1024": (1024, 2816, ((8, 8, 128), (16, 4, 64)), (16, 4, 64)),
+             "w2048": (2048, 5632, ((16, 16, 128), (32, 4, 64)), (32, 4, 64)),
+             "w4096": (4096, 14336, ((32, 16, 128), (32, 8, 128)), (32, 8, 128))}
+    WINDOW, CHUNK, TAPS = 1024, 2048, 4
+    ORDER = ("delta", "attention", "delta", "attention_2")
+    KINDS = ORDER[:2] + ORDER[3:]              # the table: all layers of one type
+
+    def own_config(self, size, layers, kind=None):
+        width, ff, ((dh, dkv, dd), (h, kv, d)), _ = self.SIZES[size]
+        mixers = {"delta": {"heads": dh, "kv_heads": dkv, "dim": dd, "vdim": dd, "conv": self.TAPS},
+                  "attention": {"heads": h, "kv_heads": kv, "dim": d, "vdim": d, "scale": d ** -0.5, "mask": {"size": self.WINDOW}},
+                  "attention_2": {"heads": h, "kv_heads": kv, "dim": d, "vdim": d, "scale": d ** -0.5, "mask": {"size": self.CHUNK},
+                                  "rot": {"base": 500000.0, "dims": d, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}}
+        return {"architecture": "Vofusun", "width": width, "vocab": self.VOCAB, "norm": {"eps": 1e-6}, "embedding": {"scale": width ** 0.5},
+                "layers": [{"type": t, "mixer": mixers[t], "mlp": {"kind": "dense", "ff": ff}}
+                           for t in ([kind] * layers if kind else [self.ORDER[i % 4] for i in range(layers)])]}
+
+    @staticmethod
+    def own_shapes(cfg):
+        D = cfg["width"]
+        out = {"final.norm": (D,), "embed": (cfg["vocab"], D)}
+        for i, L in enumerate(cfg["layers"]):
+            m, p, ff = L["mixer"], f"l{i}.", L["mlp"]["ff"]
+            H, G, d, e = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            out.update({p + "norm1": (D,), p + "norm2": (D,), p + "mlp.gate": (ff, D), p + "mlp.up": (ff, D), p + "mlp.down": (D, ff), p + "mix.o": (D, H * e)})
+            if L["type"] == "delta":
+                for n, rows in (("q", G * d), ("k", G * d), ("v", H * e)):
+                    out.update({p + f"mix.{n}": (rows, D), p + f"mix.{n}.conv": (rows, m["conv"])})
+                out.update({p + "mix.a": (H, D), p + "mix.b": (H, D), p + "mix.A_log": (H,), p + "mix.dt_bias": (H,), p + "mix.norm": (e,), p + "mix.g": (H * e, D)})
+            else:
+                out.update({p + "mix.q": (H * d, D), p + "mix.k": (G * d, D)})
+                out.update({p + "mix.v": (G * e, D)} if L["type"] == "attention" else {p + "mix.g": (H * e, D)})
+        return out
+
+    def config(self, world):
+        return {**super().config(world), "workload": "decoder with delta-rule and masked-attention layers (Vofusun) in the runtime", "layer": self.CFG["layers"][:4]}
+
+    def extra(self):
+        import statistics as st
+        tt = [t[0] for t in self.timings[-5:]]; dd = [t[1] for t in self.timings[-5:]]
+        ms_tok = st.median(dd) / max(1, self.NEW - 1)
+        step = self.weight_bytes + 2 * self.VOCAB * self.CFG["width"]                       # the head is the embedding table
+        for L in self.CFG["layers"]:                                                        # state read and written; keys and values read
+            m = L["mixer"]
+            step += self.B * (m["heads"] * m["dim"] * m["vdim"] * 8 if L["type"] == "delta" else (self.T + self.NEW // 2) * m["kv_heads"] * (m["dim"] + m["vdim"]) * 2)
+        return {"ttft_ms": st.median(tt), "decode_ms_per_token": ms_tok, "decode_step_bytes": step, "decode_hbm_GBs": step / (ms_tok * 1e-3) / 1e9,
+                "gemm_calls_total": self.sess.gemm_calls}
+
+    def cpu_run(self, orc, n, threads, reps=1):
+        """n = new tokens; prompt 32.  Four random layers, run as a loop, stand for all of them."""
+        import numpy as np
+        from oracle import hybrid_ref as hr
+        if not hasattr(self, "_cpu_w"):
+            cfg = dict(self.own_config("w2048", 4), loop={"start": 0, "stop": 4, "times": self.LAYERS // 4})
+            rng = np.random.default_rng(5)
+            self._cpu_w = (cfg, {k: (np.ones(s) if "norm" in k else rng.standard_normal(s, dtype=np.float32) * 0.02) for k, s in self.own_shapes(cfg).items()})
+        ids = list(np.random.default_rng(1).integers(0, self.VOCAB, 32))
+        t0 = time.perf_counter()
+        for _ in range(reps):
+            seq = list(ids)
+            for _ in range(n):
+                seq.append(int(np.argmax(hr.forward(*self._cpu_w, seq)[-1])))
+        dt = (time.perf_counter() - t0) / reps
+        return n / dt, dt
 
 
 # --------------------------------------------------------------------------------------
@@ -1103,7 +1178,7 @@ class WaveApi:
 
 
 WORKLOADS = {"wave_api": WaveApi, "fa_steps": FaSteps, "segops": SegopsSweep, "decode": DecodeGQA, "prefill": PrefillCausal, "decode_long": DecodeLong,
-             "runtime": RuntimeLlama, "runtime_latent": RuntimeLatent}
+             "runtime": RuntimeLlama, "runtime_latent": RuntimeLatent, "runtime_hybrid": RuntimeHybrid}
 ALL_ORDER = ["prefill", "decode", "segops", "decode_long", "runtime", "fa_steps", "wave_api"]   # `--workload all`: the first is the headline
 
 
