@@ -186,7 +186,7 @@ struct HybridState {
     bool looped = false;
     // activations of the current scratch
     void *norm = nullptr, *proj = nullptr, *q = nullptr, *attn = nullptr, *act = nullptr;
-    float *ab = nullptr, *proj32 = nullptr, *gu = nullptr, *kq = nullptr, *v = nullptr, *gb = nullptr, *o = nullptr;
+    float *ab = nullptr, *proj32 = nullptr, *gu = nullptr, *rows = nullptr, *cols = nullptr, *o = nullptr;
 };
 HybridState* hybrid(const b200p_session* s) { return static_cast<HybridState*>(s->decoder.get()); }
 
@@ -231,7 +231,7 @@ DeltaArgs delta_args(const b200p_session* s, size_t pass, int Tn, int pos0, cons
     a.eps = s->eps; a.proj = L->proj; a.ldp = a.d.main_row(); a.ab = L->ab; a.ld_ab = a.d.ab_row();
     a.conv = w.conv; a.a_log = w.a_log; a.dt_bias = w.dt_bias; a.norm = w.head_norm;
     a.state = L->kept[pass].state; a.ring = L->kept[pass].ring;
-    a.kq = L->kq; a.v = L->v; a.gb = L->gb; a.o = L->o; a.out = L->attn;
+    a.rows = L->rows; a.cols = L->cols; a.o = L->o; a.out = L->attn;
     a.abort_word = s->d_attn_status;
     return a;
 }
@@ -367,14 +367,13 @@ int hybrid_alloc_scratch(b200p_session* s, int M) {
     if ((c = s->alloc_scratch(&L->act, m * L->max_ff * e))) return int(c);
     if ((c = s->alloc_scratch(&L->gu, m * 2 * L->max_ff * 4))) return int(c);
     if (L->looped) if ((c = s->alloc_scratch(&s->embedded, m * L->H * 4))) return int(c);
-    DeltaScratch n{0, 0, 0, 0};
+    DeltaScratch n{0, 0, 0};
     for (const HybridLayer& l : L->spec.layers)
         if (l.type->delta) {
             const DeltaScratch x = delta_scratch(l.delta(), s->batch, M);
-            n = {std::max(n.kq, x.kq), std::max(n.v, x.v), std::max(n.gb, x.gb), std::max(n.o, x.o)};
+            n = {std::max(n.rows, x.rows), std::max(n.cols, x.cols), std::max(n.o, x.o)};
         }
-    if ((c = s->alloc_scratch(&L->kq, n.kq * 4)) || (c = s->alloc_scratch(&L->v, n.v * 4)) || (c = s->alloc_scratch(&L->gb, n.gb * 4)) ||
-        (c = s->alloc_scratch(&L->o, n.o * 4))) return int(c);
+    if ((c = s->alloc_scratch(&L->rows, n.rows * 4)) || (c = s->alloc_scratch(&L->cols, n.cols * 4)) || (c = s->alloc_scratch(&L->o, n.o * 4))) return int(c);
     return B200P_OK;
 }
 

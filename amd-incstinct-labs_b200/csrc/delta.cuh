@@ -7,14 +7,16 @@
 // q, k and v come out of a projection through a causal convolution per channel and silu; o is
 // divided by its root mean square over vdim, scaled by a weight and gated by silu.
 //
-// Many tokens go in blocks of sixteen: with G_t the product of the block's decays up to t and
-// R_it = G_t / G_i (kept as products of decays, never as a quotient),
+// Many tokens go in blocks of sixteen.  With G_t the product of the block's decays up to t, R_it that of
+// the decays between i and t (products of decays, never a quotient) and S0 the state ahead of the block,
 //     u_t = beta_t (v_t - G_t S0^T k_t - sum_{i<t} R_it (k_i.k_t) u_i)
 //     o_t = G_t S0^T q_t + sum_{i<=t} R_it (k_i.q_t) u_i
-//     S   = G_16 S0 + sum_i R_i16 k_i u_i^T
-// so the products with S0 and the update are small matrix products, and only a 16 x 16
-// triangle is sequential.  Everything past the convolutions is fp32 arithmetic (packed fp32x2
-// FMAs): a tensor-core form would need three passes per product to keep fp32 accuracy.
+// Solving the triangle for u (T = (1 + L)^-1 diag(beta), L_ti = beta_t R_it k_i.k_t) and putting it into
+// o (M_ti = R_it k_i.q_t) leaves everything that depends on the block alone to be computed for all blocks
+// at once, and a step from block to block without a triangle:
+//     u = T V - (T G K) S0,   o = M T V + (G Q - M T G K) S0,   S = G_16 S0 + sum_i R_i16 k_i u_i^T
+// Everything past the convolutions is fp32 arithmetic (packed fp32x2 FMAs): a tensor-core form would
+// need three passes per product to keep fp32 accuracy.
 //
 // Sizes are padded with zero columns: dim and vdim to multiples of 16 in the projection, the
 // rows of S to a multiple of 32.
@@ -32,15 +34,14 @@ struct DeltaDims {
     int taps;                      // of the convolutions, the current token's included
     __host__ __device__ int group() const { return heads / kv_heads; }
     __host__ __device__ int rows() const { return (dim + 31) / 32 * 32; }                  // of S
-    __host__ __device__ int slices() const { return (vdim + 63) / 64; }                    // 64-column slices of v
     __host__ __device__ int channels() const { return 2 * kv_heads * dim + heads * vdim; } // with a convolution: [q | k | v]
     __host__ __device__ int g_col() const { return channels(); }
     __host__ __device__ int v_row() const { return heads * vdim; }
     __host__ __device__ int main_row() const { return channels() + heads * vdim; }         // [q | k | v | gate]
     __host__ __device__ int ab_row() const { return (2 * heads + 15) / 16 * 16; }          // [decay inputs | step inputs], always fp32
     __host__ __device__ size_t state_floats() const { return size_t(heads) * rows() * vdim; }
-    // one block of sixteen tokens of a query/key head: k, q [16][rows], (k_i.k_t), (k_i.q_t) [16 i][16 t]
-    __host__ __device__ int kq_block() const { return 32 * rows() + 512; }
+    // one block of sixteen tokens of a head: [16][rows] of T G K, of G Q - M T G K and of R_i16 k_i, then G_16
+    __host__ __device__ int row_block() const { return 48 * rows() + 4; }
 };
 constexpr int kDeltaBlock = 16;
 
@@ -59,9 +60,8 @@ struct DeltaArgs {
     float* state;                  // [batch][heads][rows][vdim]; position 0 starts from zero whatever it holds
     float* ring;                   // [batch][taps][channels]: the convolutions' input at position p is in slot p % taps
     // many tokens only: blocks = ceil(Tn / 16)
-    float* kq;                     // [batch][kv_heads][blocks][kq_block]
-    float* v;                      // [batch][heads][slices][blocks][16][64]
-    float* gb;                     // [batch][heads][blocks][32]: decays, steps
+    float* rows;                   // [batch][heads][blocks][row_block]
+    float* cols;                   // [batch][heads][vdim / 16][blocks][2][16 tokens][16 columns]: T V, M T V
     float* o;                      // [batch * Tn][v_row]
     void* out;                     // [batch * Tn][v_row]: normalised and gated, of type dtype
     int* abort_word;
@@ -74,10 +74,10 @@ bool delta_step_ok(const DeltaDims& d);
 int delta_step(const DeltaArgs& a, cudaStream_t st);
 
 // Floats of the buffers for up to M tokens of all sequences.
-struct DeltaScratch { size_t kq, v, gb, o; };
+struct DeltaScratch { size_t rows, cols, o; };
 inline DeltaScratch delta_scratch(const DeltaDims& d, int batch, int M) {
     const size_t blocks = (size_t(M) + size_t(batch) * (kDeltaBlock - 1)) / kDeltaBlock;        // every sequence may end in a partial one
-    return {blocks * d.kv_heads * d.kq_block(), blocks * d.heads * d.slices() * 1024, blocks * d.heads * 32, size_t(M) * d.v_row()};
+    return {blocks * d.heads * d.row_block(), blocks * d.heads * d.vdim * 32, size_t(M) * d.v_row()};
 }
 
 } // namespace b200p
