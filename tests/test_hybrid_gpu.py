@@ -409,6 +409,18 @@ def test_plain_and_fast_kernels_agree(opened, knob, name, key):
         check(fast, plain.astype(np.float64), dtype)
 
 
+@pytest.mark.parametrize("columns", [1, 2, 4])
+@pytest.mark.parametrize("name", ["odd", "real_heads", "unequal", "no_scaling"])
+def test_forms_of_the_block_walk(opened, knob, name, columns):
+    """The delta rule's blocks with and without tensor cores, whatever the columns are dealt to."""
+    ids = tokens(CONFIGS[name], 150)
+    knob("delta_columns", columns)
+    for dtype, tensor in (("bf16", 1), ("bf16", 0), ("f32", 1)):
+        knob("delta_tensor", tensor)
+        s = opened(name, dtype)
+        check(run(s, ids, [100, 20, 2, 1]), reference(name, ids), dtype, (tensor, columns))
+
+
 @pytest.mark.parametrize("name,dtype,batch", [("odd", "bf16", 2), ("odd", "f32", 1), ("real_heads", "bf16", 1), ("too_wide", "bf16", 1)])
 def test_greedy_generation(opened, name, dtype, batch):
     """generate() (the greedy loop, replayed as a graph where the step can be captured): the tokens of the host-driven loop
