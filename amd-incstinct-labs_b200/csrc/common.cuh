@@ -38,7 +38,7 @@ enum Knob {
     KNOB_LATENT_PLAIN,          // 1: latent attention of 16-bit sessions on the plain kernel as well
     KNOB_GROUPED_PLAIN,         // 1: grouped attention of 16-bit sessions on the plain kernel as well
     KNOB_DELTA_PLAIN,           // 1: the gated delta rule token by token on the plain kernel
-    KNOB_DELTA_COLUMNS,         // 1, 2 or 4: columns of S per lane (tensor-core form: 16-column slices per CTA) in the walk over blocks
+    KNOB_DELTA_COLUMNS,         // 1, 2 or 4: columns of S per lane (tensor-core form: 4, 2 or 1 warps per 16 columns) in the walk over blocks
     KNOB_DELTA_TENSOR,          // 0: blocks of 16-bit sessions without tensor cores as well
     KNOB_COUNT
 };
