@@ -182,10 +182,10 @@ struct HybridState {
     HybridSpec spec;
     std::vector<HybridWeights> w;                      // by layer
     std::vector<PassState> kept;                       // by pass
-    int H = 0, max_ff = 0, max_main = 0, max_ab = 0, max_q = 0, max_v = 0;
+    int H = 0, max_ff = 0, max_main = 0, max_ab = 0, max_v = 0;
     bool looped = false;
     // activations of the current scratch
-    void *norm = nullptr, *proj = nullptr, *q = nullptr, *attn = nullptr, *act = nullptr;
+    void *norm = nullptr, *proj = nullptr, *attn = nullptr, *act = nullptr;
     float *ab = nullptr, *proj32 = nullptr, *gu = nullptr, *rows = nullptr, *cols = nullptr, *o = nullptr;
 };
 HybridState* hybrid(const b200p_session* s) { return static_cast<HybridState*>(s->decoder.get()); }
@@ -216,7 +216,7 @@ GroupedAttn grouped_args(const b200p_session* s, size_t pass, int Tn, int pos0, 
     a.dtype = s->dtype; a.batch = s->batch; a.Tn = Tn; a.pos0 = pos0; a.max_seq = s->max_seq; a.pos_dev = pos_dev;
     a.scale = float(ly.scale); a.eps = s->eps; a.norm = ly.type->normed; a.plus_one = ly.type->plus_one;
     a.cos_t = w.rot.first; a.sin_t = w.rot.second;
-    a.proj = L->proj; a.q = L->q; a.kcache = L->kept[pass].k; a.vcache = L->kept[pass].v; a.out = L->attn;
+    a.proj = L->proj; a.kcache = L->kept[pass].k; a.vcache = L->kept[pass].v; a.out = L->attn;
     a.abort_word = s->d_attn_status;
     return a;
 }
@@ -362,7 +362,6 @@ int hybrid_alloc_scratch(b200p_session* s, int M) {
     if ((c = s->alloc_scratch(&L->proj, m * L->max_main * e))) return int(c);
     if ((c = s->alloc_scratch(&L->ab, m * L->max_ab * 4))) return int(c);
     if ((c = s->alloc_scratch(&L->proj32, std::min<size_t>(m, kSkinnyMaxM) * (L->max_main + L->max_ab) * 4))) return int(c);
-    if ((c = s->alloc_scratch(&L->q, m * L->max_q * e))) return int(c);
     if ((c = s->alloc_scratch(&L->attn, m * L->max_v * e))) return int(c);
     if ((c = s->alloc_scratch(&L->act, m * L->max_ff * e))) return int(c);
     if ((c = s->alloc_scratch(&L->gu, m * 2 * L->max_ff * 4))) return int(c);
@@ -480,7 +479,6 @@ int hybrid_build(b200p_session* s, const b200p_model* m) {
     for (const HybridLayer& ly : L->spec.layers) {
         L->max_ff = std::max(L->max_ff, pad16(ly.ff)); L->max_main = std::max(L->max_main, ly.main_row()); L->max_ab = std::max(L->max_ab, ly.ab_row());
         L->max_v = std::max(L->max_v, ly.v_row());
-        if (!ly.type->delta) L->max_q = std::max(L->max_q, ly.grouped().q_row());
     }
     for (const HybridSpec::Pass& p : L->spec.passes) L->looped = L->looped || p.embed_again;
     if (int rc = s->dtype == B200P_F32 ? build_weights<float>(s, m) : build_weights<__nv_bfloat16>(s, m)) return rc;

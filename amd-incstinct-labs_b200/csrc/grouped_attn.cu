@@ -42,46 +42,78 @@ __device__ __forceinline__ float4 rotate_quad(const float4& v, const GroupedAttn
 __device__ __forceinline__ float dot4(const float4& x, const float4& y) { return (x.x * y.x + x.y * y.y) + (x.z * y.z + x.w * y.w); }
 __device__ __forceinline__ float4 scaled(const float4& v, float f) { return make_float4(v.x * f, v.y * f, v.z * f, v.w * f); }
 
-// One warp per (token, head): query heads to q, key heads to the cache (and the values, own or the keys as projected).
-constexpr int kHeadQuads = 4;            // quads per lane held in registers: heads up to 512 columns
-template <typename T>
-__global__ void __launch_bounds__(256) grouped_inputs_kernel(const GroupedAttn a) {
+// A group of W lanes per (token, head), eight columns a lane: key heads to the cache (and the values, own or the keys as
+// projected); query heads, where something happens to them, in place.
+template <typename T, int W, int CH>
+__global__ void __launch_bounds__(256) grouped_inputs_kernel(const GroupedAttn a, unsigned units, int slots) {
     const GroupedDims& d = a.d;
-    const int slots = d.heads + d.kv_heads;
-    const size_t j = size_t(blockIdx.x) * 8 + threadIdx.x / 32;
-    const int lane = threadIdx.x % 32;
-    if (j >= size_t(a.batch) * a.Tn * slots) return;
-    const size_t row = j / slots;
-    const int slot = int(j % slots), b = int(row / a.Tn), pos = a.pos0 + int(row % a.Tn);
-    const bool is_k = slot >= d.heads;
-    const int kvh = slot - d.heads;
-    const T* p = static_cast<const T*>(a.proj) + row * d.proj_row();
-    const T* src = p + size_t(slot) * d.dim;
-    float4 v[kHeadQuads];
+    const unsigned u = (blockIdx.x * 256u + threadIdx.x) / W;
+    const int c0 = threadIdx.x % W * 8;
+    const bool live = u < units;
+    const unsigned row = (live ? u : 0) / unsigned(slots);
+    const int slot = int((live ? u : 0) - row * slots) + (d.heads + d.kv_heads - slots);          // without queries: the keys only
+    const unsigned b = row / unsigned(a.Tn);
+    const int pos = a.pos0 + int(row - b * a.Tn), kvh = slot - d.heads;
+    T* p = static_cast<T*>(const_cast<void*>(a.proj)) + size_t(row) * d.proj_row();
+    T* src = p + slot * d.dim;
+    const size_t cache_row = (size_t(b) * d.kv_heads + kvh) * a.max_seq + pos;
+    T* dst = kvh >= 0 ? static_cast<T*>(a.kcache) + cache_row * d.dim : src;
+    T* vrow = static_cast<T*>(a.vcache) + cache_row * d.vdim;
+    float v[CH][8];
     float ss = 0.f;
     #pragma unroll
-    for (int i = 0; i < kHeadQuads; ++i) {
-        const int col = 4 * (lane + 32 * i);
-        if (col < d.dim) { v[i] = load4<T>(src + col); ss += dot4(v[i], v[i]); }
-    }
-    const size_t cache_row = (size_t(b) * d.kv_heads + kvh) * a.max_seq + pos;
-    if (is_k) {
-        T* vrow = static_cast<T*>(a.vcache) + cache_row * d.vdim;
-        if (d.own_values) {
-            for (int col = 4 * lane; col < d.vdim; col += 128) store4<T>(vrow + col, load4<T>(p + d.v_col() + size_t(kvh) * d.vdim + col));
-        } else {
+    for (int i = 0; i < CH; ++i) {
+        const int c = c0 + 8 * W * i;
+        if (live && c < d.dim) {
+            load8<T>(src + c, v[i]);
             #pragma unroll
-            for (int i = 0; i < kHeadQuads; ++i) if (4 * (lane + 32 * i) < d.dim) store4<T>(vrow + 4 * (lane + 32 * i), v[i]);
+            for (int k = 0; k < 8; ++k) ss += v[i][k] * v[i][k];
+            if (kvh >= 0 && !d.own_values) store8<T>(vrow + c, v[i]);
         }
     }
+    if (live && kvh >= 0 && d.own_values)
+        for (int c = c0; c < d.vdim; c += 8 * W) {
+            float x[8];
+            load8<T>(p + d.v_col() + kvh * d.vdim + c, x);
+            store8<T>(vrow + c, x);
+        }
     // (turning a pair does not change its length: the mean square is the same before and after)
-    const float f = a.norm ? rsqrtf(wave::dpp::reduce_sum(ss) / d.n_dim + a.eps) : 1.f;
-    T* dst = is_k ? static_cast<T*>(a.kcache) + cache_row * d.dim : static_cast<T*>(a.q) + row * d.q_row() + size_t(slot) * d.dim;
+    const float f = a.norm ? rsqrtf(wave::lane_group_reduce<W>(ss, wave::SumOp{}) / d.n_dim + a.eps) : 1.f;
     #pragma unroll
-    for (int i = 0; i < kHeadQuads; ++i) {
-        const int col = 4 * (lane + 32 * i);
-        if (col < d.dim) store4<T>(dst + col, scaled(a.cos_t ? rotate_quad(v[i], a, pos, col) : v[i], f));
+    for (int i = 0; i < CH; ++i) {
+        const int c = c0 + 8 * W * i;
+        if (!live || c >= d.dim) continue;
+        if (a.cos_t) {
+            const size_t t = size_t(pos) * (d.dim / 2) + c / 2;
+            const float4 cs = load4<float>(a.cos_t + t), sn = load4<float>(a.sin_t + t);
+            const float cf[4] = {cs.x, cs.y, cs.z, cs.w}, sf[4] = {sn.x, sn.y, sn.z, sn.w};
+            #pragma unroll
+            for (int k = 0; k < 4; ++k) {
+                const float x = v[i][2 * k], y = v[i][2 * k + 1];
+                v[i][2 * k] = x * cf[k] - y * sf[k];
+                v[i][2 * k + 1] = y * cf[k] + x * sf[k];
+            }
+        }
+        #pragma unroll
+        for (int k = 0; k < 8; ++k) v[i][k] *= f;
+        store8<T>(dst + c, v[i]);
     }
+}
+
+template <typename T>
+int launch_inputs(const GroupedAttn& a, cudaStream_t st) {
+    const int slots = (a.cos_t || a.norm ? a.d.heads : 0) + a.d.kv_heads, lanes = a.d.dim / 8;
+    const long long units = (long long)a.batch * a.Tn * slots;
+    if (units * 32 > 0xffffffffLL) return B200P_E_RANGE;
+    auto run = [&](auto kern, int W) {
+        kern<<<unsigned((units * W + 255) / 256), 256, 0, st>>>(a, unsigned(units), slots);
+        return launched();
+    };
+    if (lanes <= 2) return run(grouped_inputs_kernel<T, 2, 1>, 2);
+    if (lanes <= 4) return run(grouped_inputs_kernel<T, 4, 1>, 4);
+    if (lanes <= 8) return run(grouped_inputs_kernel<T, 8, 1>, 8);
+    if (lanes <= 16) return run(grouped_inputs_kernel<T, 16, 1>, 16);
+    return run(grouped_inputs_kernel<T, 32, 2>, 32);
 }
 
 // ---- any shape, fp32 arithmetic ---------------------------------------------------------------------------
@@ -100,7 +132,7 @@ __global__ void __launch_bounds__(kPlainRows * 32) grouped_plain_kernel(const Gr
     const int h = blockIdx.y, b = blockIdx.z, t0 = blockIdx.x * kPlainRows, t = t0 + warp;
     const bool live = t < a.Tn;
     const size_t row = size_t(b) * a.Tn + (live ? t : 0);
-    const T* q = static_cast<const T*>(a.q) + row * d.q_row() + size_t(h) * DT;
+    const T* q = static_cast<const T*>(a.proj) + row * d.proj_row() + size_t(h) * DT;
     for (int i = lane; i < DT; i += 32) sq[warp * DT + i] = live ? to_float(q[i]) : 0.f;
     const int last = a.pos0 + t, first = a.mask.first(last);                 // keys this row sees
     const int end = a.pos0 + min(t0 + kPlainRows, a.Tn);                     // keys any row of the CTA sees: [begin, end)
@@ -429,12 +461,8 @@ int launch_step(const GroupedAttn& a, cudaStream_t st) {
 } // namespace
 
 int grouped_inputs(const GroupedAttn& a, cudaStream_t st) {
-    if (a.d.dim > 128 * kHeadQuads || a.d.vdim > 128 * kHeadQuads) return B200P_E_DIM;
-    const size_t warps = size_t(a.batch) * a.Tn * (a.d.heads + a.d.kv_heads);
-    const unsigned grid = unsigned((warps + 7) / 8);
-    if (a.dtype == B200P_F32) grouped_inputs_kernel<float><<<grid, 256, 0, st>>>(a);
-    else grouped_inputs_kernel<T16><<<grid, 256, 0, st>>>(a);
-    return launched();
+    if (a.d.dim > 512 || a.d.vdim > 512) return B200P_E_DIM;
+    return a.dtype == B200P_F32 ? launch_inputs<float>(a, st) : launch_inputs<T16>(a, st);
 }
 
 int grouped_plain(const GroupedAttn& a, cudaStream_t st) {

@@ -8,7 +8,7 @@
 // Head sizes are padded to multiples of 16 with zero columns (the session packs the weights
 // that way), so every row is TMA shaped whatever the model's sizes are.
 //
-//   grouped_inputs   a projection's rows -> queries, and keys and values into the cache
+//   grouped_inputs   a projection's rows: queries turned and normalised in place, keys and values into the cache
 //   grouped_plain    any shape and type, fp32 arithmetic
 //   grouped_prefill  many query rows: the tcgen05 kernel (prefill_tc.cuh)
 //   grouped_step     one new token per sequence: one launch from the projection's fp32 rows to the
@@ -27,7 +27,6 @@ struct GroupedDims {
     int n_dim;                     // query/key columns without padding: what the norm's mean is over
     bool own_values, gated;        // values of their own / the keys as projected; output gate
     __host__ __device__ int group() const { return heads / kv_heads; }
-    __host__ __device__ int q_row() const { return heads * dim; }
     __host__ __device__ int v_row() const { return heads * vdim; }
     // the projection: [queries | keys | values of their own | gate]
     __host__ __device__ int k_col() const { return heads * dim; }
@@ -45,8 +44,7 @@ struct GroupedAttn {
     float scale, eps;
     bool norm, plus_one;           // queries and keys by their root mean square; e^0 joins the denominator
     const float *cos_t, *sin_t;    // [max_seq][dim / 2] (1 and 0 where nothing turns), or null: no positions
-    const void* proj;              // [batch * Tn][proj_row]: the session's type; grouped_step: fp32
-    void* q;                       // [batch * Tn][q_row]
+    const void* proj;              // [batch * Tn][proj_row]: the session's type; grouped_step: fp32.  grouped_inputs leaves the queries in it
     void *kcache, *vcache;         // [batch][kv_heads][max_seq][dim], [..][vdim]
     void* out;                     // [batch * Tn][v_row]
     int* abort_word;               // grouped_step: raised by a wait that gives up
