@@ -414,14 +414,14 @@ __global__ void __launch_bounds__(kBlockThreads) delta_blocks_kernel(const Delta
 // ---- many tokens on the tensor cores (16-bit sessions) ----------------------------------------------------------
 // The same two kernels with their products as mma_fp32.  Rows of k and q (and of the block form's first two matrices)
 // are 64 bytes longer than S's: a quarter-warp's 16-byte reads of two rows fall on different banks.
+constexpr int kMatLd = 20;              // floats between the rows of a 16 x 16 matrix: 16-byte reads of eight rows on different banks
 struct PrepMma {
-    float kk[256], kq[256];            // (k_i.k_t), (k_i.q_t) at [i][t], before the unit lengths
-    float l[256], m[256];              // the triangles of u and o at [t][i]
-    float t_[256];                     // T at [j][t]
-    float coef[4][16 * 20];            // [t][20 j]: T, M T, and both times G_j / |k_j|
+    float kk[16 * kMatLd], kq[16 * kMatLd];        // (k_i.k_t), (k_i.q_t) at [t][i], before the unit lengths
+    float l[16 * kMatLd], m[16 * kMatLd];          // the triangles of u and o at [t][i]
+    float t_[256];                                 // T at [j][t]
+    float coef[4][16 * kMatLd];                    // [t][j]: T, M T, and both times G_j / |k_j|
     float g[16], beta[16], G[16], tail[16], rk[16], rq[16];
 };
-constexpr int kCoefLd = 20;
 
 template <typename P, int TAPS, int X>
 __global__ void __launch_bounds__(256, 3) delta_prepare_mma_kernel(const DeltaArgs a) {
@@ -429,7 +429,7 @@ __global__ void __launch_bounds__(256, 3) delta_prepare_mma_kernel(const DeltaAr
     __shared__ __align__(16) PrepMma x;
     constexpr int R = 16 * X, ld = R + 16;
     const DeltaDims& d = a.d;
-    const int ldv = d.vdim + 16;
+    const int ldv = d.vdim + 8;
     float *ks = prep_smem, *qs = ks + kDeltaBlock * ld, *vs = qs + kDeltaBlock * ld;
     const int blk = blockIdx.x, nblk = gridDim.x, kvh = blockIdx.y, b = blockIdx.z, t0 = blk * kDeltaBlock;
     const int tid = threadIdx.x, warp = tid / 32, lane = tid % 32, r = lane / 4, q = lane % 4;
@@ -457,7 +457,7 @@ __global__ void __launch_bounds__(256, 3) delta_prepare_mma_kernel(const DeltaAr
         }
         float* dots = of_q ? x.kq : x.kk;
         #pragma unroll
-        for (int e = 0; e < 4; ++e) dots[(i0 + 2 * q + (e & 1)) * 16 + r + 8 * (e >> 1)] = acc[0][e] + acc[1][e];
+        for (int e = 0; e < 4; ++e) dots[(r + 8 * (e >> 1)) * kMatLd + i0 + 2 * q + (e & 1)] = acc[0][e] + acc[1][e];
     } else {
         const float q_scale = rsqrtf(float(d.n_dim));
         float ss[8];                                              // unit lengths: warps 4, 5 the keys, 6, 7 the queries
@@ -487,8 +487,8 @@ __global__ void __launch_bounds__(256, 3) delta_prepare_mma_kernel(const DeltaAr
             float f = t > i ? x.g[t] : 1.f;                       // the decays between i and t: a running product over the 16 lanes
             #pragma unroll
             for (int y = 1; y < 16; y *= 2) { const float o = __shfl_up_sync(0xffffffffu, f, y, 16); if (t >= y) f *= o; }
-            x.l[t * 16 + i] = t > i ? x.beta[t] * f * x.kk[i * 16 + t] * x.rk[i] * x.rk[t] : 0.f;
-            x.m[t * 16 + i] = t >= i ? f * x.kq[i * 16 + t] * x.rk[i] * x.rq[t] : 0.f;
+            x.l[t * kMatLd + i] = t > i ? x.beta[t] * f * x.kk[t * kMatLd + i] * x.rk[i] * x.rk[t] : 0.f;
+            x.m[t * kMatLd + i] = t >= i ? f * x.kq[t * kMatLd + i] * x.rk[i] * x.rq[t] : 0.f;
             if (t == 15) x.tail[i] = f * x.rk[i];
             if (i == 0) x.G[t] = f * x.g[0];
         }
@@ -503,7 +503,7 @@ __global__ void __launch_bounds__(256, 3) delta_prepare_mma_kernel(const DeltaAr
                 float s = t == j ? x.beta[t] : 0.f;
                 #pragma unroll
                 for (int i4 = 0; i4 < t; i4 += 4) {
-                    const float4 f = load4<float>(&x.l[t * 16 + i4]);
+                    const float4 f = load4<float>(&x.l[t * kMatLd + i4]);
                     s -= f.x * c[i4];
                     if (i4 + 1 < t) s -= f.y * c[i4 + 1];
                     if (i4 + 2 < t) s -= f.z * c[i4 + 2];
@@ -532,10 +532,10 @@ __global__ void __launch_bounds__(256, 3) delta_prepare_mma_kernel(const DeltaAr
             const int j = tid / 16, t = tid % 16;
             float s = 0.f;
             #pragma unroll
-            for (int i = 0; i < 16; i += 4) s += dot4(load4<float>(&x.m[t * 16 + i]), load4<float>(&x.t_[j * 16 + i]));
+            for (int i = 0; i < 16; i += 4) s += dot4(load4<float>(&x.m[t * kMatLd + i]), load4<float>(&x.t_[j * 16 + i]));
             const float f = x.G[j] * x.rk[j], T = x.t_[tid];
-            x.coef[0][t * kCoefLd + j] = T; x.coef[1][t * kCoefLd + j] = s;
-            x.coef[2][t * kCoefLd + j] = T * f; x.coef[3][t * kCoefLd + j] = s * f;
+            x.coef[0][t * kMatLd + j] = T; x.coef[1][t * kMatLd + j] = s;
+            x.coef[2][t * kMatLd + j] = T * f; x.coef[3][t * kMatLd + j] = s * f;
         }
         __syncthreads();
         // A fragments of two of the 16 x 16 matrices: k-steps j = q, q + 4 and q + 8, q + 12
@@ -545,7 +545,7 @@ __global__ void __launch_bounds__(256, 3) delta_prepare_mma_kernel(const DeltaAr
             for (int y = 0; y < 2; ++y)
                 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
-                    const int at = (r + 8 * (e & 1)) * kCoefLd + 8 * y + q + 4 * (e >> 1);
+                    const int at = (r + 8 * (e & 1)) * kMatLd + 8 * y + q + 4 * (e >> 1);
                     f0[y][e] = split(x.coef[which][at]); f1[y][e] = split(x.coef[which + 1][at]);
                 }
         };
@@ -988,7 +988,7 @@ int launch_blocks_mma(const DeltaArgs& a, cudaStream_t st) {
 
 template <typename P, int X>
 int launch_prepare_mma_x(const DeltaArgs& a, int nblk, cudaStream_t st) {
-    const size_t smem = size_t(kDeltaBlock) * (2 * (16 * X + 16) + a.d.vdim + 16) * 4;
+    const size_t smem = size_t(kDeltaBlock) * (2 * (16 * X + 16) + a.d.vdim + 8) * 4;
     auto kern = a.d.taps == 4 ? delta_prepare_mma_kernel<P, 4, X> : delta_prepare_mma_kernel<P, 0, X>;
     if (smem > 36 * 1024)
         if (cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem))) return int(e);

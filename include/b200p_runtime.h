@@ -92,7 +92,7 @@ b200p_session* b200p_session_create(const b200p_model_weights* weights, int max_
 void b200p_session_destroy(b200p_session* s);
 /* The same for any model, whatever its architecture.  dtype: compute type, B200P_BF16 / B200P_F16 / B200P_F32, or -1 for
  * the model's own.  B200P_E_DTYPE where the decoder has no kernels of that type (B200P_F32, true 32-bit throughout:
- * Maposun only). */
+ * the decoders of config.json models only). */
 b200p_session* b200p_session_open(const b200p_model* model, int dtype, int max_seq, int batch, int* status);
 
 /* Session::generate (session.hpp:263-296): greedy decoding.
@@ -115,8 +115,9 @@ int b200p_session_step_logits(b200p_session* s, const int* token_ids, float* log
 
 /* The next T tokens of every sequence on top of the current cache: a whole prompt, a portion of one, or one token.
  * input_ids: host, [batch, T].  want: host, n_want indexes among the T tokens whose logits are asked for (may be none);
- * logits: host, fp32 [batch, n_want, vocab].  b200p_session_reset gives the cache back: the next tokens start new
- * sequences. */
+ * logits: host, fp32 [batch, n_want, vocab].  b200p_session_reset gives the cache (and any recurrent state) back: the
+ * next tokens start new sequences.  After a call that failed on the device (not one whose arguments were refused) a
+ * recurrent state may have moved on: reset the session before its next tokens. */
 int b200p_session_extend(b200p_session* s, const int* input_ids, int T, const int* want, int n_want, float* logits,
                          b200p_stream_t stream);
 void b200p_session_reset(b200p_session* s);

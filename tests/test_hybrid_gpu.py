@@ -276,6 +276,21 @@ def test_key_splits_of_the_step(opened, knob, splits):
         check(run(s, ids[:20], [1]), reference(name, ids[:20]), "bf16", name)
 
 
+@pytest.mark.parametrize("dtype,splits", [("f32", 0), ("bf16", 0), ("bf16", 1), ("bf16", 2)])
+def test_masks_of_many_key_tiles(opened, knob, dtype, splits):
+    """Windows and chunks of about a thousand keys: every ring of key tiles goes round more than once, in prompts and in
+    decoding."""
+    cfg = config(96, 90, [window(4, 2, 64, 48, 1000), window(2, 1, 128, 112, 900), chunk(2, 1, 32, 1040, 32, scale=0.3), delta(2, 2, 32, 32, 4)])
+    name = "long"
+    ids = tokens(cfg, 1150, 16)
+    want = reference(name, ids, cfg)
+    if splits:
+        knob("decode_splits", splits)
+    s = opened(name, dtype, max_seq=1150, cfg=cfg)
+    for portions in ([1150], [1030, 1], [600, 300, 130, 2]):
+        check(run(s, ids, portions), want, dtype, portions)
+
+
 # ---- memories ----------------------------------------------------------------------------------------------------------
 def memory_model(name, a_log, dt_bias, taps=4):
     cfg = config(96, 120, [delta(4, 2, 40, 72, taps), delta(2, 2, 64, 32, taps)])
