@@ -9,8 +9,8 @@
 //                   registers, the rows come through a ring of bulk copies;
 //   delta_finish    norm and gate, and the convolutions' last inputs.
 // Preparation and walk come in two forms.  16-bit sessions run the products on the tensor cores
-// (the _mma kernels): three tf32 passes per product with fp32 accumulation, which loses a few 2^-22 of a
-// product.  fp32 sessions run them as packed fp32x2 FMAs: S over 8 lanes x rows / 8 with 1 to 4 columns
+// (the _mma kernels): three tf32 passes per product with fp32 accumulation, relative error of a product
+// about 2^-21.  fp32 sessions run them as packed fp32x2 FMAs: S over 8 lanes x rows / 8 with 1 to 4 columns
 // per lane, eight sums at a time reduced and scattered over the eight lanes in seven shuffles; a lane's
 // loads from shared memory, one word per column and FMA, bound that form.
 // One token: delta_step, a cluster per (sequence, head), 32 columns of S per CTA; S and the
